@@ -12,6 +12,7 @@ from .registry import (
     load_config,
     register_architecture,
 )
+from .sorizen import SorizenConfig
 from .tepavik import TepavikConfig
 from .specs import LayerSpec, ModelSpec, PartSpec, ScheduleEntry, TensorSpec
 
@@ -20,6 +21,7 @@ register_architecture(TepavikConfig)
 register_architecture(BomipelConfig)
 register_architecture(KanavikConfig)
 register_architecture(RekodraConfig)
+register_architecture(SorizenConfig)
 
 __all__ = [
     "BomipelConfig",
@@ -33,6 +35,7 @@ __all__ = [
     "Qwen2Config",
     "RekodraConfig",
     "ScheduleEntry",
+    "SorizenConfig",
     "TensorSpec",
     "TepavikConfig",
     "config_class_for",

@@ -82,8 +82,13 @@ class ModelSpec:
     schedule: tuple[ScheduleEntry, ...]
     final_norm: PartSpec
     head: PartSpec
+    #: number of residual streams of a model whose blocks read and write several of them through
+    #: vectors of their own (None: one stream that every sublayer's output is added to)
+    streams: int | None = None
 
     def __post_init__(self) -> None:
+        if self.streams is not None and any(entry.add_embedding for entry in self.schedule):
+            raise ValueError("a model of several residual streams does not add its embedding output again")
         for index, entry in enumerate(self.schedule):
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(

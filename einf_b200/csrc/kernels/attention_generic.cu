@@ -18,7 +18,8 @@
 // z * tanh(s / z) before the softmax.  Keys and values may have different sizes per head.
 // With `keep_first` n > 0 a windowed token also sees the first n positions of its sequence
 // (j < n), at their true positions.  With `sink` (one float per query head) the softmax's
-// denominator of head h also holds exp(sink[h]): a column with no key and no value, unscaled.
+// denominator of head h also holds exp(sink[h]): a column with no key and no value, unscaled.  With
+// `gate` (one float per token and query head) a head's mixed row is multiplied by it before it is rounded.
 // `value_stride` is the distance between two value rows in
 // elements: value_size for a cache of its own, the key size when the values are the leading
 // elements of the key rows (a latent cache that holds one row per token for both).
@@ -56,7 +57,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
                                T* __restrict__ out, int num_rows, int num_heads, int num_kv_heads,
                                int head_size, int value_size, int value_stride, int page_size, int num_pages,
                                int table_width, float scale, int window, int keep_first, int chunk, float softcap,
-                               const float* __restrict__ sink, int* status) {
+                               const float* __restrict__ sink, const float* __restrict__ gate, int* status) {
   __shared__ float q_smem[kWarpsPerBlock][kHeadLimit];
   pdl_launch_dependents();
   pdl_wait();
@@ -150,6 +151,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
     const float keys = (m == -INFINITY) ? 0.f : l * expf(m - top);
     inv = (m == -INFINITY) ? 0.f : expf(m - top) / (keys + expf(s - top));
   }
+  if (gate) inv *= gate[row];
   T* o_row = out + (size_t)row * value_size;
 #pragma unroll
   for (int i = 0; i < kDimsPerLane; ++i) {
@@ -168,9 +170,22 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
 // scores and a stripe of value dimensions for the mixing.  The shares of a token's keys (grid x)
 // leave unnormalised (accumulator, maximum, sum) triples in a workspace, which a second kernel
 // adds up in share order; with one share the CTA writes the result itself.
-// Arithmetic and order of additions are 32-bit and fixed per (token, head): nothing depends on
-// what else the batch holds.
+// With a window the shares cut its keys; a sink joins the denominator once, where the shares meet, and so
+// does a gate (see above).  Arithmetic and order of additions are 32-bit and fixed per (token, head): nothing
+// depends on what else the batch holds.
 // ---------------------------------------------------------------------------
+// What an accumulator with maximum m and sum l is multiplied by at the end: one over the sum, to which the head's
+// sink adds (against the larger of the two maxima), times the gate.
+__device__ __forceinline__ float final_factor(float m, float l, const float* __restrict__ sink,
+                                              const float* __restrict__ gate, int head, size_t row) {
+  float factor = l > 0.f ? 1.f / l : 0.f;
+  if (sink && m != -INFINITY) {
+    const float top = fmaxf(m, sink[head]);
+    factor = expf(m - top) / (l * expf(m - top) + expf(sink[head] - top));
+  }
+  return gate ? factor * gate[row] : factor;
+}
+
 constexpr int kSharedWarps = 8;
 constexpr int kSharedHeads = 2 * kSharedWarps;   // heads a CTA takes
 constexpr int kSharedTile = 32;                  // keys per tile
@@ -181,7 +196,8 @@ latent_decode_attention_kernel(const T* __restrict__ q, const T* __restrict__ ca
                                const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                                T* __restrict__ out, float* __restrict__ part_acc, float* __restrict__ part_ml,
                                int num_heads, int row_size, int value_size, int page_size, int num_pages,
-                               int table_width, float scale, int* status) {
+                               int table_width, float scale, int window, const float* __restrict__ sink,
+                               const float* __restrict__ gate, int* status) {
   extern __shared__ __align__(16) unsigned char shared_raw[];
   // rows start on 16-byte borders, 16 bytes off a multiple of the row's own length
   const int row_pad = (row_size + 16 / (int)sizeof(T) - 1) / (16 / (int)sizeof(T)) * (16 / (int)sizeof(T)) + 16 / (int)sizeof(T);
@@ -195,9 +211,10 @@ latent_decode_attention_kernel(const T* __restrict__ q, const T* __restrict__ ca
   const int heads_here = min(kSharedHeads, num_heads - head0);
   const int pos = positions[t];
   const int* table = block_table + (size_t)seq_of_token[t] * table_width;
-  int per = (pos + 1 + splits - 1) / splits;
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  int per = (pos + 1 - lo + splits - 1) / splits;
   per = (per + kSharedTile - 1) / kSharedTile * kSharedTile;
-  const int k_begin = min(pos + 1, split * per), k_end = min(pos + 1, k_begin + per);
+  const int k_begin = min(pos + 1, lo + split * per), k_end = min(pos + 1, k_begin + per);
 
   for (int i = threadIdx.x; i < heads_here * row_size; i += blockDim.x) {
     const int h = i / row_size, d = i - h * row_size;
@@ -303,7 +320,7 @@ latent_decode_attention_kernel(const T* __restrict__ q, const T* __restrict__ ca
   auto finish = [&](int h, const float* acc, float m, float l) {
     const int head = head0 + h;
     if (splits == 1) {
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = final_factor(m, l, sink, gate, head, (size_t)t * num_heads + head);
       T* o = out + ((size_t)t * num_heads + head) * value_size;
 #pragma unroll
       for (int i = 0; i < kDimsPerLane; ++i) {
@@ -328,10 +345,11 @@ latent_decode_attention_kernel(const T* __restrict__ q, const T* __restrict__ ca
   if (has_b) finish(h_b, acc_b, m_b, l_b);
 }
 
-// out[t, h] = sum_s w_s acc_s / sum_s w_s l_s with w_s = exp(m_s - max m), the shares in order.
+// out[t, h] = sum_s w_s acc_s / sum_s w_s l_s with w_s = exp(m_s - max m), the shares in order (then sink and gate).
 template <typename T>
 __global__ void latent_decode_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                           T* __restrict__ out, int splits, int value_size) {
+                                           T* __restrict__ out, int splits, int value_size, int num_heads,
+                                           const float* __restrict__ sink, const float* __restrict__ gate) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t row = blockIdx.x;
@@ -340,7 +358,7 @@ __global__ void latent_decode_merge_kernel(const float* __restrict__ part_acc, c
   for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[2 * s]);
   float l = 0.f;
   for (int s = 0; s < splits; ++s) l += ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - m) * ml[2 * s + 1];
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = final_factor(m, l, sink, gate, (int)(row % num_heads), row);
   for (int d = threadIdx.x; d < value_size; d += blockDim.x) {
     float v = 0.f;
     for (int s = 0; s < splits; ++s)
@@ -359,7 +377,7 @@ extern "C" int einf_paged_attention_generic(const void* q, const void* k_cache, 
                                             int num_heads, int num_kv_heads, int head_size, int value_size,
                                             int value_stride, int page_size, int num_pages, int table_width,
                                             float scale, int window, int keep_first, int chunk, float softcap,
-                                            const float* sink, int* status, cudaStream_t stream) {
+                                            const float* sink, const float* gate, int* status, cudaStream_t stream) {
   const int rows = num_tokens * num_heads;
   if (rows == 0) return 0;
   if (head_size > kMaxHeadSize || value_size > kMaxHeadSize || head_size <= 0 || value_size <= 0)
@@ -371,12 +389,12 @@ extern "C" int einf_paged_attention_generic(const void* q, const void* k_cache, 
       paged_attention_generic_kernel<T, 256><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
           (const T*)q, (const T*)k_cache, (const T*)v_cache, block_table, seq_of_token, positions, (T*)out,
           rows, num_heads, num_kv_heads, head_size, value_size, value_stride, page_size, num_pages, table_width,
-          scale, window, keep_first, chunk, softcap, sink, status);
+          scale, window, keep_first, chunk, softcap, sink, gate, status);
     } else {
       paged_attention_generic_kernel<T, kMaxHeadSize><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
           (const T*)q, (const T*)k_cache, (const T*)v_cache, block_table, seq_of_token, positions, (T*)out,
           rows, num_heads, num_kv_heads, head_size, value_size, value_stride, page_size, num_pages, table_width,
-          scale, window, keep_first, chunk, softcap, sink, status);
+          scale, window, keep_first, chunk, softcap, sink, gate, status);
     }
   })
   return (int)cudaGetLastError();
@@ -390,8 +408,8 @@ extern "C" int einf_latent_decode_attention(const void* q, const void* cache, in
                                             const int* seq_of_token, const int* positions, void* out,
                                             float* part_acc, float* part_ml, int num_tokens, int num_heads,
                                             int row_size, int value_size, int page_size, int num_pages,
-                                            int table_width, float scale, int splits, int* status,
-                                            cudaStream_t stream) {
+                                            int table_width, float scale, int splits, int window, const float* sink,
+                                            const float* gate, int* status, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (row_size <= 0 || row_size > kMaxHeadSize || value_size <= 0 || value_size > row_size || splits < 1 ||
       (splits > 1 && (!part_acc || !part_ml)) || num_tokens > 65535)
@@ -409,11 +427,12 @@ extern "C" int einf_latent_decode_attention(const void* q, const void* cache, in
     if (e != cudaSuccess) return (int)e;
     e = launch_pdl(kernel, grid, dim3(kSharedWarps * 32), smem, stream, (const T*)q, (const T*)cache, block_table,
                    seq_of_token, positions, (T*)out, part_acc, part_ml, num_heads, row_size, value_size, page_size,
-                   num_pages, table_width, scale, status);
+                   num_pages, table_width, scale, window, sink, gate, status);
     if (e != cudaSuccess) return (int)e;
     if (splits > 1)
       e = launch_pdl(latent_decode_merge_kernel<T>, dim3(num_tokens * num_heads), dim3(128), 0, stream,
-                     (const float*)part_acc, (const float*)part_ml, (T*)out, splits, value_size);
+                     (const float*)part_acc, (const float*)part_ml, (T*)out, splits, value_size, num_heads,
+                     sink, gate);
   })
   return (int)e;
 }

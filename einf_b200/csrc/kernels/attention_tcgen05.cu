@@ -366,6 +366,7 @@ struct TcAttentionParams {
   int chunk;                // chunked mask: a row sees only the keys of its own block of this many positions (0: off)
   float scale, softcap;     // scores are multiplied by scale; with a cap z they become z * tanh(score / z)
   const float* sink;        // [heads] or null: exp(sink[h]) joins the denominator of head h, with no key and no value
+  const float* gate;        // [tokens, heads] or null: a head's mixed row is multiplied by it before it is rounded
 };
 
 __global__ void __launch_bounds__(kAttnThreads, 1)
@@ -857,7 +858,8 @@ paged_prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q
     // for a cluster: this CTA's share (sums of both warpgroups, not yet divided), after the exchange area
     float* part_o = reinterpret_cast<float*>(gbase + kShareOff);
     float* part_ml = part_o + kBlockQ * (D + 1);
-    const float inv = csize > 1 ? 1.f : (l_all > 0.f ? 1.f / l_all : 0.f);
+    float inv = csize > 1 ? 1.f : (l_all > 0.f ? 1.f / l_all : 0.f);
+    if (p.gate && csize == 1 && pos >= 0) inv *= p.gate[(size_t)(token0 + r) * p.num_heads + head];
     __nv_bfloat16* dst = p.out + ((size_t)(token0 + r) * p.num_heads + head) * D + g * kDimsHere;
 #pragma unroll 1
     for (int c0 = 0; c0 < kDimsHere; c0 += 32) {
@@ -917,7 +919,8 @@ paged_prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q
       for (int offset = 4; offset >= 1; offset >>= 1) l += __shfl_xor_sync(0xffffffffu, l, offset);
       l = __shfl_sync(0xffffffffu, l, 0);
       if (p.sink && m != -INFINITY) l += exp2f(p.sink[head] * 1.4426950408889634f - m);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate) inv *= p.gate[(size_t)(token0 + row) * p.num_heads + head];
       float o[D / 32];
 #pragma unroll
       for (int j = 0; j < D / 32; ++j) o[j] = 0.f;
@@ -988,6 +991,7 @@ struct TcDecodeParams {
   int chunk;                // see TcAttentionParams
   float scale, softcap;
   const float* sink;        // see TcAttentionParams
+  const float* gate;        // see TcAttentionParams
   // A token's keys split over `splits` clusters, which meet in global memory: every cluster writes its
   // unnormalised share [16 heads][D + 2] (the accumulator, then maximum and sum) to split_out, every
   // CTA counts itself in split_count, and the CTA that finds itself the last adds the shares up.
@@ -1383,6 +1387,7 @@ paged_decode_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
     }
     if (!kSplit) {
       if (p.sink && m != -INFINITY) l += exp2f(p.sink[first_head + row] * 1.4426950408889634f - m);
+      if (p.gate) o *= p.gate[token_heads + first_head + row];
       p.out[(token_heads + first_head + row) * D + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     } else {
       float* share = p.split_out + (((size_t)pair * p.splits + split) * kDecHeads + row) * (D + 2);
@@ -1435,6 +1440,7 @@ paged_decode_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
         o += oc[c] * f;
       }
       if (p.sink && m != -INFINITY) l += exp2f(p.sink[first_head + row] * 1.4426950408889634f - m);
+      if (p.gate) o *= p.gate[token_heads + first_head + row];
       p.out[(token_heads + first_head + row) * D + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     }
   }
@@ -1530,7 +1536,8 @@ extern "C" int einf_paged_prefill_attention_tcgen05(const void* q, const void* k
                                                     void* out, int num_tokens, int num_heads, int num_kv_heads,
                                                     int page_size, int num_pages, int table_width, float scale,
                                                     int window, int keep_first, int chunk, float softcap, int cluster,
-                                                    const float* sink, int* status, cudaStream_t stream) {
+                                                    const float* sink, const float* gate, int* status,
+                                                    cudaStream_t stream) {
   if (num_tiles == 0) return 0;
   if (cluster < 1 || cluster > 8) return (int)cudaErrorInvalidValue;
   if (keep_first < 0 || (keep_first > 0 && window > 0 && cluster != 1)) return (int)cudaErrorInvalidValue;
@@ -1564,6 +1571,7 @@ extern "C" int einf_paged_prefill_attention_tcgen05(const void* q, const void* k
   p.scale = scale;
   p.softcap = softcap;
   p.sink = sink;
+  p.gate = gate;
   cudaError_t e = cudaFuncSetAttribute(paged_prefill_attention_tcgen05_kernel,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
   if (e != cudaSuccess) return (int)e;
@@ -1631,7 +1639,7 @@ extern "C" int einf_paged_decode_attention_tcgen05(const void* q, const void* k_
                                                    int num_tokens, int num_heads, int num_kv_heads, int page_size,
                                                    int num_pages, int table_width, float scale, int window,
                                                    int keep_first, int chunk, float softcap, int cluster, int splits,
-                                                   float* split_out, int* split_count, const float* sink,
+                                                   float* split_out, int* split_count, const float* sink, const float* gate,
                                                    int* status, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (cluster < 1 || cluster > kDecMaxCluster) return (int)cudaErrorInvalidValue;
@@ -1667,6 +1675,7 @@ extern "C" int einf_paged_decode_attention_tcgen05(const void* q, const void* k_
   p.scale = scale;
   p.softcap = softcap;
   p.sink = sink;
+  p.gate = gate;
   p.splits = splits;
   p.split_out = split_out;
   p.split_count = split_count;

@@ -771,6 +771,7 @@ __global__ void zero_fresh_state_kernel(Word* __restrict__ state, long long row_
 //   1 GELU, tanh form   0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 //   2 SiLU              z / (1 + exp(-z))
 //   3 ReLU
+//   4 GELU, exact      0.5 z (1 + erf(z / sqrt(2)))
 // x may be the float32 partial sums of a split-K product.
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ float activate(float z, int kind) {
@@ -778,6 +779,7 @@ __device__ __forceinline__ float activate(float z, int kind) {
     case 0: { const float r = fmaxf(z, 0.f); return r * r; }
     case 1: return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
     case 2: return z / (1.f + expf(-z));
+    case 4: return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
     default: return fmaxf(z, 0.f);
   }
 }
@@ -1619,7 +1621,7 @@ extern "C" int einf_zero_fresh_state(void* state, long long row_bytes, int num_s
 extern "C" int einf_activation(const void* x, int in_dtype, int splits, long long split_stride, void* out, int dtype,
                                long long total, int kind, cudaStream_t stream) {
   if (total <= 0) return 0;
-  if (kind < 0 || kind > 3) return (int)cudaErrorInvalidValue;
+  if (kind < 0 || kind > 4) return (int)cudaErrorInvalidValue;
   const int threads = 256;
   if (splits == 1 && in_dtype == kBFloat16 && dtype == kBFloat16 && total % 8 == 0 && ((uintptr_t)x & 15) == 0 &&
       ((uintptr_t)out & 15) == 0) {

@@ -3,10 +3,10 @@
 //
 //   einf_router_topk   per token: the `top_k` largest router logits (ties to the lower index),
 //                      their weights sigmoid(z) or softmax(z) over all experts, optionally
-//                      divided by their sum; 32-bit throughout.  With a correction the choice goes
+//                      divided by their sum (plus a constant) and multiplied by another; 32-bit throughout.  With a correction the choice goes
 //                      by score + correction (the weights stay the scores); with groups only the
-//                      experts of the `keep` groups of neighbours whose best choice score is
-//                      largest can be chosen
+//                      experts of the `keep` groups of neighbours whose best choice score (or
+//                      the sum of whose two best) is largest can be chosen
 //   einf_moe_dispatch  counts per expert, offsets (experts in order), the place of every
 //                      (token, choice) in the order sorted by expert, and the rows gathered into
 //                      that order (times the router weight where the weight acts on the input);
@@ -34,8 +34,9 @@ constexpr int kMaxExpertsPerLane = 32;   // experts up to 1024
 
 __global__ void router_topk_kernel(const float* __restrict__ logits, int splits, size_t split_stride, int num_tokens,
                                    int row_width, int num_experts, int top_k, int score, int renormalise,
-                                   const float* __restrict__ correction, int group_count, int group_keep,
-                                   int* __restrict__ expert_ids, float* __restrict__ weights) {
+                                   float renormalise_eps, float weight_scale, const float* __restrict__ correction,
+                                   int group_count, int group_keep, int group_best, int* __restrict__ expert_ids,
+                                   float* __restrict__ weights) {
   // per warp of the CTA: [num_experts] what the choice goes by | [num_experts] the scores (with a correction) |
   // [group_count] 1 for a group that may be chosen from
   extern __shared__ float z_all[];
@@ -73,8 +74,12 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int splits,
     }
     __syncwarp();
   }
+  auto choice_score = [&](float v) {
+    if (correction) return v;
+    return score == kScoreSoftmax ? expf(v - z_max) / denominator : 1.f / (1.f + expf(-v));
+  };
   if (group_count > 0) {
-    // a group's score is its best choice score; the `group_keep` best groups stay open (ties to the lower index)
+    // a group's score is its best choice score, or the sum of its two best; the `group_keep` best groups stay open (ties to the lower index)
     const int per_group = num_experts / group_count;
     for (int g = lane; g < group_count; g += 32) group_open[g] = 0.f;
     __syncwarp();
@@ -83,8 +88,17 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int splits,
       int best_g = 0x7fffffff;
       for (int g = lane; g < group_count; g += 32) {
         if (group_open[g] != 0.f) continue;
-        float top = -INFINITY;
-        for (int i = 0; i < per_group; ++i) top = fmaxf(top, z[g * per_group + i]);
+        float top = -INFINITY, second = -INFINITY;
+        for (int i = 0; i < per_group; ++i) {
+          const float v = z[g * per_group + i];
+          second = fmaxf(second, fminf(top, v));
+          top = fmaxf(top, v);
+        }
+        if (group_best == 2) {
+          // sums are of scores: without a correction z still holds the logits (ordered as the scores are)
+          top = choice_score(top);
+          if (per_group > 1) top += choice_score(second);
+        }
         if (top > best || best_g == 0x7fffffff) {
           best = top;
           best_g = g;
@@ -136,8 +150,12 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int splits,
       weights[(size_t)t * top_k + j] = w;
     }
   }
-  if (renormalise && lane == 0) {
-    for (int j = 0; j < top_k; ++j) weights[(size_t)t * top_k + j] /= chosen_sum;
+  if ((renormalise || weight_scale != 1.f) && lane == 0) {
+    for (int j = 0; j < top_k; ++j) {
+      float w = weights[(size_t)t * top_k + j];
+      if (renormalise) w /= chosen_sum + renormalise_eps;
+      weights[(size_t)t * top_k + j] = w * weight_scale;
+    }
   }
 }
 
@@ -410,8 +428,8 @@ using namespace einf;
 
 extern "C" int einf_router_topk(const float* logits, int splits, long long split_stride, int num_tokens,
                                 int row_width, int num_experts, int top_k, int score, int renormalise,
-                                const float* correction, int group_count, int group_keep, int* expert_ids,
-                                float* weights, cudaStream_t stream) {
+                                float renormalise_eps, float weight_scale, const float* correction, int group_count,
+                                int group_keep, int group_best, int* expert_ids, float* weights, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (num_experts <= 0 || num_experts > 32 * kMaxExpertsPerLane || top_k <= 0 || top_k > num_experts ||
       row_width < num_experts)
@@ -424,7 +442,8 @@ extern "C" int einf_router_topk(const float* logits, int splits, long long split
   const size_t per_warp = (size_t)(correction ? 2 : 1) * num_experts + group_count;
   return (int)launch_pdl(router_topk_kernel, blocks, threads, (size_t)(threads / 32) * per_warp * sizeof(float), stream,
                          logits, splits < 1 ? 1 : splits, (size_t)split_stride, num_tokens, row_width, num_experts, top_k,
-                         score, renormalise, correction, group_count, group_keep, expert_ids, weights);
+                         score, renormalise, renormalise_eps, weight_scale, correction, group_count, group_keep,
+                         group_best, expert_ids, weights);
 }
 
 // x: [T, hidden]; expert_ids, weights, place: [T * top_k]; work: [3 E + 1] int32 (offsets are its last

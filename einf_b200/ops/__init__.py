@@ -526,6 +526,11 @@ def project(
     return out
 
 
+def _check_gate(gate: Optional[torch.Tensor], tokens: int, heads: int) -> None:
+    if gate is not None and (gate.dtype != torch.float32 or gate.shape != (tokens, heads)):
+        raise ValueError(f"gate must be float32 {(tokens, heads)}, got {gate.dtype} {tuple(gate.shape)}")
+
+
 def paged_attention_generic(
     q: torch.Tensor,
     k_cache: torch.Tensor,
@@ -542,6 +547,7 @@ def paged_attention_generic(
     keep_first: int = 0,
     values_in_keys: Optional[int] = None,
     sink: Optional[torch.Tensor] = None,
+    gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Causal attention of every token of the batch over the pages of its request.
 
@@ -554,11 +560,13 @@ def paged_attention_generic(
     ``z * tanh(score / z)`` before the softmax.  ``values_in_keys`` n (with ``v_cache`` None): a
     token's value is the first n elements of its key row (one cached row serves as both).
     ``sink`` (float32 ``[heads]``): the softmax's denominator of head h also holds ``exp(sink[h])``,
-    unscaled, with no key and no value.
+    unscaled, with no key and no value.  ``gate`` (float32 ``[tokens, heads]``): a head's mixed row is multiplied
+    by it before it is rounded.
     """
     tokens, num_heads, head_size = q.shape
     if sink is not None and (sink.dtype != torch.float32 or sink.shape != (num_heads,)):
         raise ValueError(f"sink must be float32 [{num_heads}]")
+    _check_gate(gate, tokens, num_heads)
     num_pages, num_kv_heads, page_size, size = k_cache.shape
     if values_in_keys is not None:
         if v_cache is not None or not 0 < values_in_keys <= size:
@@ -582,7 +590,8 @@ def paged_attention_generic(
     fn = _fn(
         "einf_paged_attention_generic",
         [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p],
+         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
+         c_void_p],
     )
     _check(
         fn(_dev(q, "q"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), _code(q),
@@ -590,7 +599,8 @@ def paged_attention_generic(
            _opt(positions, "positions", torch.int32), _dev(out, "out"), tokens, num_heads, num_kv_heads,
            head_size, value_size, value_stride, page_size, num_pages, block_table.shape[1], float(scale),
            int(window) if window else 0, int(keep_first) if window else 0, int(chunk) if chunk else 0,
-           float(softcap) if softcap else 0.0, _opt(sink, "sink", torch.float32), _dev(status, "status"), _stream()),
+           float(softcap) if softcap else 0.0, _opt(sink, "sink", torch.float32), _opt(gate, "gate", torch.float32),
+           _dev(status, "status"), _stream()),
         "paged_attention_generic",
     )
 
@@ -620,16 +630,23 @@ def latent_decode_attention(
     scale: float,
     splits: int,
     status: torch.Tensor,
+    window: Optional[int] = None,
+    sink: Optional[torch.Tensor] = None,
+    gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Causal attention of single tokens over rows that all query heads share: ``q [tokens, heads, row]``,
     ``cache [pages, 1, page_size, row]`` whose first ``out.shape[2]`` elements are the values.  A CTA stages
     32 rows at a time in shared memory for sixteen heads; ``splits`` CTAs share a token's keys and a
-    second kernel adds their results up in order (the workspace is kept per shape)."""
+    second kernel adds their results up in order (the workspace is kept per shape).
+    ``window``, ``sink`` and ``gate``: see :func:`paged_attention_generic`."""
     tokens, heads, row = q.shape
     pages, kv_heads, page_size, size = cache.shape
     value_size = out.shape[2]
     if kv_heads != 1 or size != row or out.shape[:2] != (tokens, heads) or not 0 < value_size <= row:
         raise ValueError(f"latent_decode_attention: q {tuple(q.shape)}, cache {tuple(cache.shape)}, out {tuple(out.shape)}")
+    if sink is not None and (sink.dtype != torch.float32 or sink.shape != (heads,)):
+        raise ValueError(f"sink must be float32 [{heads}]")
+    _check_gate(gate, tokens, heads)
     if row > MAX_GENERIC_HEAD_SIZE:
         raise UnsupportedSize(f"rows up to {MAX_GENERIC_HEAD_SIZE} elements, got {row}")
     if not (q.dtype == cache.dtype == out.dtype):
@@ -650,23 +667,24 @@ def latent_decode_attention(
     fn = _fn(
         "einf_latent_decode_attention",
         [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-         c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p],
+         c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     )
     _check(
         fn(_dev(q, "q"), _dev(cache, "cache"), _code(q), _opt(block_table, "block_table", torch.int32),
            _opt(seq_of_token, "seq_of_token", torch.int32), _opt(positions, "positions", torch.int32), _dev(out, "out"),
            acc_ptr, ml_ptr, tokens, heads, row, value_size, page_size, pages, block_table.shape[1], float(scale),
-           int(splits), _dev(status, "status"), _stream()),
+           int(splits), int(window) if window else 0, _opt(sink, "sink", torch.float32),
+           _opt(gate, "gate", torch.float32), _dev(status, "status"), _stream()),
         "latent_decode_attention",
     )
 
 
 #: activations of :func:`activation` by name
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "relu": 3}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "gelu": 4}
 
 
 def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> None:
-    """``out = act(x)`` elementwise (``relu2``: the square of ReLU; ``gelu_tanh``; ``silu``; ``relu``);
+    """``out = act(x)`` elementwise (``relu2``: the square of ReLU; ``gelu_tanh``; ``silu``; ``relu``; ``gelu``: the exact form);
     ``x`` may be float32 partial sums ``[splits, tokens, width]`` of a split-K product."""
     tokens, width = out.shape
     splits, stride = _maybe_split(x, tokens, width, "x")
@@ -803,12 +821,14 @@ def latent_down_store(
     q_latent_out: Optional[torch.Tensor],
     cache: Optional[torch.Tensor],
     status: torch.Tensor,
+    amplitude: float = 1.0,
 ) -> None:
     """From a token's product row ``[query latent q_rank | kv latent kv_rank | key part rot_dim]`` (or its
     float32 split-K partial sums): the RMS-normed query latent into ``q_latent_out [tokens, q_rank]``, and
     the cache row ``[normed kv latent | rotated key part]`` into the page slot of the token (``cache``
     ``[pages, 1, page_size, kv_rank + rot_dim]``; ``slots`` None writes none).  Norms carry a weight and
-    ``eps`` inside the root; everything is computed in 32-bit and rounded once."""
+    ``eps`` inside the root, cosine and sine the factor ``amplitude``; everything is computed in 32-bit and
+    rounded once."""
     tokens = down.shape[-2]
     width = q_rank + kv_rank + rot_dim
     splits, stride = _maybe_split(down, tokens, width, "down")
@@ -829,13 +849,13 @@ def latent_down_store(
     fn = _fn(
         "einf_latent_down_store",
         [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
-         c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+         c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     )
     _check(
         fn(_dev(down, "down"), _code(down), splits, stride, _code(dtype_of), tokens, q_rank, kv_rank, rot_dim,
            _opt(q_norm_weight, "q_norm_weight", torch.float32) if q_rank else 0,
            _opt(kv_norm_weight, "kv_norm_weight", torch.float32), float(eps),
-           _opt(positions, "positions", torch.int32), _opt(inv_freq, "inv_freq", torch.float32),
+           _opt(positions, "positions", torch.int32), _opt(inv_freq, "inv_freq", torch.float32), float(amplitude),
            1 if interleaved else 0, _opt(slots, "slots", torch.int32) if cache_ptr else 0,
            _dev(q_latent_out, "q_latent_out") if q_rank else 0, cache_ptr, page_size, num_pages,
            _dev(status, "status"), _stream()),
@@ -850,6 +870,7 @@ def latent_q_store(
     interleaved: bool,
     q_plain: torch.Tensor,
     q_full: torch.Tensor,
+    amplitude: float = 1.0,
 ) -> None:
     """Queries ``[tokens, heads * (dim + rot_dim)]`` (or partial sums), head by head ``[dim plain | rot_dim
     to rotate]``: the plain part into ``q_plain [tokens, heads, dim]``, the rotated part into the last
@@ -862,14 +883,72 @@ def latent_q_store(
     splits, stride = _maybe_split(q, tokens, heads * (dim + rot_dim), "q")
     fn = _fn(
         "einf_latent_q_store",
-        [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+        [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
          c_void_p, c_void_p, c_void_p],
     )
     _check(
         fn(_dev(q, "q"), _code(q), splits, stride, _code(q_plain), tokens, heads, dim, rot_dim, kv_rank,
-           _opt(positions, "positions", torch.int32), _opt(inv_freq, "inv_freq", torch.float32),
+           _opt(positions, "positions", torch.int32), _opt(inv_freq, "inv_freq", torch.float32), float(amplitude),
            1 if interleaved else 0, _dev(q_plain, "q_plain"), _dev(q_full, "q_full"), _stream()),
         "latent_q_store",
+    )
+
+
+def latent_qkv_store(
+    product: torch.Tensor,
+    kv_rank: int,
+    rot_dim: int,
+    kv_norm_weight: torch.Tensor,
+    eps: float,
+    positions: torch.Tensor,
+    inv_freq: torch.Tensor,
+    interleaved: bool,
+    amplitude: float,
+    slots: Optional[torch.Tensor],
+    q_plain: Optional[torch.Tensor],
+    q_full: torch.Tensor,
+    gate: Optional[torch.Tensor],
+    cache: Optional[torch.Tensor],
+    status: torch.Tensor,
+    dim: int,
+) -> None:
+    """The two functions above in one launch, for queries without a latent of their own.  A row of
+    ``product`` (or of its float32 split-K partial sums) is ``[kv latent kv_rank | key part rot_dim | heads *
+    (dim plain, rot_dim to rotate)]``, with ``gate`` (float32 ``[tokens, heads]``) followed by one logit per
+    head, whose sigmoid goes there.  The cache row ``[normed latent | rotated key part | zeros]`` goes into
+    the token's page slot (``cache [pages, 1, page_size, row]``; ``slots`` None writes none), the rotated query
+    parts and zeros behind them into ``q_full [tokens, heads, row]`` from ``kv_rank`` on, the plain parts into
+    ``q_plain [tokens, heads, dim]`` (None: the caller reads them out of ``product`` itself)."""
+    tokens, heads, row = q_full.shape
+    width = kv_rank + rot_dim + heads * (dim + rot_dim) + (heads if gate is not None else 0)
+    splits, stride = _maybe_split(product, tokens, width, "product")
+    if inv_freq.shape[0] * 2 != rot_dim or row < kv_rank + rot_dim:
+        raise ValueError(f"{rot_dim} rotated dimensions need {rot_dim // 2} frequencies and rows of {kv_rank + rot_dim}")
+    if (kv_rank + 2 * rot_dim) * 4 > 48 * 1024:
+        raise UnsupportedSize(f"latent rows of {kv_rank + rot_dim} values exceed the kernel's shared memory")
+    if q_plain is not None and (q_plain.shape != (tokens, heads, dim) or q_plain.dtype != q_full.dtype):
+        raise ValueError(f"q_plain must be {(tokens, heads, dim)} of q_full's dtype")
+    if gate is not None and (gate.dtype != torch.float32 or gate.shape != (tokens, heads)):
+        raise ValueError(f"gate must be float32 {(tokens, heads)}")
+    page_size = num_pages = cache_ptr = 0
+    if slots is not None:
+        if cache is None or cache.shape[1] != 1 or cache.shape[3] != row or cache.dtype != q_full.dtype:
+            raise ValueError(f"the latent cache must be [pages, 1, page, {row}] of q_full's dtype")
+        num_pages, _, page_size, _ = cache.shape
+        cache_ptr = _dev(cache, "cache")
+    fn = _fn(
+        "einf_latent_qkv_store",
+        [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
+         c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+    )
+    _check(
+        fn(_dev(product, "product"), _code(product), splits, stride, _code(q_full), tokens, kv_rank, rot_dim, heads,
+           int(dim), row, _opt(kv_norm_weight, "kv_norm_weight", torch.float32), float(eps),
+           _opt(positions, "positions", torch.int32), _opt(inv_freq, "inv_freq", torch.float32), float(amplitude),
+           1 if interleaved else 0, _opt(slots, "slots", torch.int32) if cache_ptr else 0,
+           0 if q_plain is None else _dev(q_plain, "q_plain"), _dev(q_full, "q_full"),
+           _opt(gate, "gate", torch.float32), cache_ptr, page_size, num_pages, _dev(status, "status"), _stream()),
+        "latent_qkv_store",
     )
 
 
@@ -902,16 +981,19 @@ ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
 
 def router_topk(logits: torch.Tensor, top_k: int, score: str, renormalise: bool, expert_ids: torch.Tensor,
                 weights: torch.Tensor, num_experts: Optional[int] = None, correction: Optional[torch.Tensor] = None,
-                groups: Optional[Tuple[int, int]] = None) -> None:
+                groups: Optional[Tuple[int, int]] = None, group_best: int = 1, renormalise_eps: float = 0.0,
+                weight_scale: float = 1.0) -> None:
     """Per row of float32 ``logits [tokens, width]`` (or split-K partial sums ``[splits, tokens, width]``,
     added up here): the ``top_k`` experts with the largest scores
     (ties to the lower index) into ``expert_ids`` (int32) and their weights into ``weights`` (float32),
     both ``[tokens, top_k]``, best first.  A weight is ``sigmoid(z)`` or the softmax over all experts;
-    ``renormalise`` divides the chosen weights by their sum.  The experts are the first ``num_experts``
+    ``renormalise`` divides the chosen weights by their sum plus ``renormalise_eps``; ``weight_scale``
+    multiplies them at the end.  The experts are the first ``num_experts``
     columns of a row (default: all of them; further columns belong to someone else).  With
     ``correction`` (float32 ``[num_experts]``) the choice goes by ``score + correction`` while the weights
     stay the scores.  With ``groups = (count, keep)`` the experts form ``count`` equal groups of
-    neighbours and only those of the ``keep`` groups whose best choice score is largest can be chosen."""
+    neighbours and only those of the ``keep`` groups whose best choice score is largest can be chosen;
+    ``group_best`` 2: whose two best choice scores have the largest sum."""
     tokens, width = logits.shape[-2:]
     experts = width if num_experts is None else int(num_experts)
     splits, stride = _maybe_split(logits, tokens, width, "logits")
@@ -927,11 +1009,14 @@ def router_topk(logits: torch.Tensor, top_k: int, score: str, renormalise: bool,
     if groups is not None:
         if count <= 0 or experts % count or not 0 < keep <= count or top_k > keep * (experts // count):
             raise ValueError(f"{experts} experts in {count} groups of which {keep} are kept cannot give {top_k} choices")
-    fn = _fn("einf_router_topk", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-                                  c_int, c_void_p, c_void_p, c_void_p])
+    if group_best not in (1, 2):
+        raise ValueError(f"a group is scored by its best one or two experts, not {group_best}")
+    fn = _fn("einf_router_topk", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                                  c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
     _check(
         fn(_dev(logits, "logits"), splits, stride, tokens, width, experts, top_k, ROUTER_SCORES[score],
-           1 if renormalise else 0, _opt(correction, "correction", torch.float32), count, keep,
+           1 if renormalise else 0, float(renormalise_eps), float(weight_scale),
+           _opt(correction, "correction", torch.float32), count, keep, int(group_best),
            _dev(expert_ids, "expert_ids"), _dev(weights, "weights"), _stream()),
         "router_topk",
     )
@@ -1620,6 +1705,71 @@ def stream_tail(
     )
 
 
+#: residual streams the kernel below takes
+MAX_STREAMS = 16
+
+
+def hyper_norm(
+    pending: Optional[torch.Tensor],
+    source: torch.Tensor,
+    streams: int,
+    connection: Optional[Tuple[torch.Tensor, torch.Tensor]],
+    read: Optional[torch.Tensor],
+    dest: Optional[torch.Tensor],
+    weight: torch.Tensor,
+    bias: Optional[torch.Tensor],
+    centre: bool,
+    eps: float,
+    out: torch.Tensor,
+    rows: Optional[torch.Tensor] = None,
+) -> None:
+    """Between two sublayers of a model with several residual streams, in 32-bit: with ``connection =
+    (mix [streams, streams], write [streams])`` and y = ``pending`` (``[T, H]``, or split-K partial sums
+    ``[splits, T, H]``, added up here) ``x'_t = sum_s mix[s, t] x_s + write[t] y``; ``u = sum_t read[t] x'_t``
+    (``read`` None: the plain sum); ``out = norm(u) * weight (+ bias)``, a layer norm (``centre``: mean off,
+    then the root of the mean squared deviation) or an RMS norm, ``eps`` inside the root.  ``source`` is
+    float32 ``[streams, T, H]``, or ``[T, H]`` while all streams are equal; ``dest`` (float32 ``[streams, T,
+    H]``, or ``[T, H]`` for one stream; may be ``source`` itself) receives x'.  Without a ``connection`` the
+    one stream is plain, ``x' = x + y``, and of several streams nothing may be pending.  With ``rows`` (int32)
+    output row r is made of row ``rows[r]`` and nothing is stored."""
+    tokens, hidden = source.shape[-2:]
+    if not 1 <= streams <= MAX_STREAMS:
+        raise UnsupportedSize(f"{streams} residual streams: the kernel takes 1 to {MAX_STREAMS}")
+    if source.dtype != torch.float32 or (source.dim() == 3 and source.shape[0] != streams):
+        raise ValueError(f"source must be float32 [{streams}, tokens, hidden] or [tokens, hidden]")
+    if dest is not None and (dest.dtype != torch.float32 or dest.numel() != streams * tokens * hidden or rows is not None):
+        raise ValueError(f"dest must be float32 [{streams}, {tokens}, {hidden}], and comes without rows")
+    for name, t, shape in (("weight", weight, (hidden,)), ("bias", bias, (hidden,)), ("read", read, (streams,)),
+                           ("mix", connection and connection[0], (streams, streams)),
+                           ("write", connection and connection[1], (streams,))):
+        if t is not None and (t.dtype != torch.float32 or t.shape != shape):
+            raise ValueError(f"{name} must be float32 {shape}, got {t.dtype} {tuple(t.shape)}")
+    if connection is None and pending is not None and streams != 1:
+        raise ValueError("what is pending reaches several streams through a connection")
+    if hidden > 48_000:
+        raise UnsupportedSize(f"hyper_norm keeps a row in shared memory; width {hidden} > 48000")
+    num_rows = rows.shape[0] if rows is not None else tokens
+    if out.shape != (num_rows, hidden):
+        raise ValueError(f"out is {tuple(out.shape)}, expected {(num_rows, hidden)}")
+    splits, stride, code, ptr = 1, 0, FLOAT32, 0
+    if pending is not None:
+        splits, stride = _maybe_split(pending, tokens, hidden, "pending")
+        code, ptr = _code(pending), _dev(pending, "pending")
+    mix_ptr, write_ptr = (0, 0) if connection is None else (_dev(connection[0], "mix"), _dev(connection[1], "write"))
+    fn = _fn(
+        "einf_hyper_norm",
+        [c_void_p, c_int, c_int, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+         c_longlong, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
+    )
+    _check(
+        fn(ptr, code, splits, stride, _dev(source, "source"), tokens * hidden if source.dim() == 3 else 0, int(streams),
+           mix_ptr, write_ptr, _opt(read, "read", torch.float32), _opt(dest, "dest", torch.float32), tokens * hidden,
+           _dev(weight, "weight"), _opt(bias, "bias", torch.float32), 1 if centre else 0, float(eps), _dev(out, "out"),
+           _code(out), _opt(rows, "rows", torch.int32), num_rows, hidden, _stream()),
+        "hyper_norm",
+    )
+
+
 # ---------------------------------------------------------------------------
 # Attention whose heads' scores meet before the softmax
 MIXED_MAX_HEADS = 32
@@ -2122,6 +2272,7 @@ def paged_decode_attention_auto(
     softcap: Optional[float] = None,
     keep_first: int = 0,
     sink: Optional[torch.Tensor] = None,
+    gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Decode attention by the kernel, cluster size and number of clusters per token that
     ``decode_plan`` picks for this batch; ``max_context`` is the longest context among the
@@ -2135,10 +2286,10 @@ def paged_decode_attention_auto(
     if kernel == "tcgen05":
         paged_decode_attention_tcgen05(q, k_cache, v_cache, block_table, seq_of_token, positions, out, scale, window,
                                        cluster, status, token_list, splits, chunk=chunk, softcap=softcap,
-                                       keep_first=keep_first, sink=sink)
-    elif chunk or softcap or (window and keep_first) or sink is not None:
-        raise UnsupportedSize("a chunked mask, a soft cap, kept first positions or a sink need the tcgen05 decode "
-                              "kernel (head size 64 or 128)")
+                                       keep_first=keep_first, sink=sink, gate=gate)
+    elif chunk or softcap or (window and keep_first) or sink is not None or gate is not None:
+        raise UnsupportedSize("a chunked mask, a soft cap, kept first positions, a sink or a gate need the tcgen05 "
+                              "decode kernel (head size 64 or 128)")
     else:
         paged_decode_attention_cluster(q, k_cache, v_cache, block_table, seq_of_token, positions, out, scale, window,
                                        cluster, status, token_list)
@@ -2226,6 +2377,7 @@ def paged_decode_attention_tcgen05(
     softcap: Optional[float] = None,
     keep_first: int = 0,
     sink: Optional[torch.Tensor] = None,
+    gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Decode attention on the tcgen05 tensor cores with the keys as the 128-row operand
     (S^T = K Q^T, O^T = V^T P^T), so the tile is full at any number of query heads.  Key splits
@@ -2241,6 +2393,7 @@ def paged_decode_attention_tcgen05(
         )
     if sink is not None and (sink.dtype != torch.float32 or sink.shape != (num_heads,)):
         raise ValueError(f"sink must be float32 [{num_heads}]")
+    _check_gate(gate, tokens, num_heads)
     if token_list is not None:
         tokens = token_list.shape[0]
     if not 1 <= cluster <= 16:
@@ -2254,7 +2407,7 @@ def paged_decode_attention_tcgen05(
     fn = _fn(
         "einf_paged_decode_attention_tcgen05",
         [c_void_p] * 8 + [c_int] * 6 + [c_float, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
-         c_void_p, c_void_p],
+         c_void_p, c_void_p, c_void_p],
         f"HEAD_SIZE={head_size}",
     )
     _check(
@@ -2266,7 +2419,7 @@ def paged_decode_attention_tcgen05(
            int(keep_first) if window else 0,
            int(chunk) if chunk else 0, float(softcap) if softcap else 0.0, cluster,
            splits, shares.data_ptr() if splits > 1 else None, counters.data_ptr() if splits > 1 else None,
-           _opt(sink, "sink", torch.float32), _dev(status, "status"), _stream()),
+           _opt(sink, "sink", torch.float32), _opt(gate, "gate", torch.float32), _dev(status, "status"), _stream()),
         "paged_decode_attention_tcgen05",
     )
 
@@ -2329,6 +2482,7 @@ def paged_prefill_attention(
     softcap: Optional[float] = None,
     keep_first: int = 0,
     sink: Optional[torch.Tensor] = None,
+    gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Tensor-core causal attention for prompt portions.  ``q_tiles`` is int32 ``[tiles, 4]``:
     request, first token (packed index), rows (at most ``Q_TILE``), position of the first row.
@@ -2338,11 +2492,12 @@ def paged_prefill_attention(
     ``mma.sync`` kernel.  ``prefill_cluster`` (1 to 8; 0: ``prefill_cluster_size`` of the number of
     row tiles and ``cached_before``, the most tokens that a portion of this step finds in the
     cache, if the caller knows it) is the number of CTAs that share a row tile's keys in the
-    tcgen05 kernel.  ``chunk``, ``softcap`` and ``sink`` (see :func:`paged_attention_generic`) are the tcgen05
+    tcgen05 kernel.  ``chunk``, ``softcap``, ``sink`` and ``gate`` (see :func:`paged_attention_generic`) are the tcgen05
     kernel's alone."""
     tokens, num_heads, head_size, num_pages, num_kv_heads, page_size = _check_fast_attention(q, k_cache, v_cache, out)
     if sink is not None and (sink.dtype != torch.float32 or sink.shape != (num_heads,)):
         raise ValueError(f"sink must be float32 [{num_heads}]")
+    _check_gate(gate, tokens, num_heads)
     if q_tiles.dtype != torch.int32 or q_tiles.dim() != 2 or q_tiles.shape[1] != 4:
         raise ValueError("q_tiles must be int32 [tiles, 4]")
     can = has_tcgen05_attention(head_size, page_size)
@@ -2357,7 +2512,7 @@ def paged_prefill_attention(
         fn = _fn(
             "einf_paged_prefill_attention_tcgen05",
             [c_void_p] * 5 + [c_int, c_void_p] + [c_int] * 6 + [c_float, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                                                                 c_void_p, c_void_p],
+                                                                 c_void_p, c_void_p, c_void_p],
             f"HEAD_SIZE={head_size}",
         )
         cluster = prefill_cluster
@@ -2375,13 +2530,13 @@ def paged_prefill_attention(
                float(scale), int(window) if window else 0, int(keep_first) if window else 0,
                int(chunk) if chunk else 0,
                float(softcap) if softcap else 0.0, int(cluster), _opt(sink, "sink", torch.float32),
-               _dev(status, "status"), _stream()),
+               _opt(gate, "gate", torch.float32), _dev(status, "status"), _stream()),
             "paged_prefill_attention_tcgen05",
         )
         return
-    if chunk or softcap or (window and keep_first) or sink is not None:
-        raise UnsupportedSize("a chunked mask, a soft cap, kept first positions or a sink need the tcgen05 prefill "
-                              "kernel (head size 64 or 128)")
+    if chunk or softcap or (window and keep_first) or sink is not None or gate is not None:
+        raise UnsupportedSize("a chunked mask, a soft cap, kept first positions, a sink or a gate need the tcgen05 "
+                              "prefill kernel (head size 64 or 128)")
     fn = _fn(
         "einf_paged_prefill_attention",
         [c_void_p] * 5 + [c_int, c_void_p] + [c_int] * 5 + [c_float, c_int, c_void_p, c_void_p],

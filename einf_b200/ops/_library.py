@@ -39,6 +39,7 @@ LAUNCHERS = {
     "einf_paged_decode_attention_tcgen05_max_clusters": "attention_tcgen05",
     "einf_latent_down_store": "latent",
     "einf_latent_q_store": "latent",
+    "einf_latent_qkv_store": "latent",
     "einf_router_topk": "routed",
     "einf_moe_dispatch": "routed",
     "einf_moe_gemm": "routed",
@@ -47,6 +48,7 @@ LAUNCHERS = {
     "einf_act_mul": "pointwise",
     "einf_norm_conv": "stream",
     "einf_stream_tail": "stream",
+    "einf_hyper_norm": "hyper",
     "einf_paged_attention_mixed": "attention_mixed",
     "einf_paged_attention_mixed_tiled": "attention_mixed_tiled",
     "einf_paged_attention_mixed_tiled_rows": "attention_mixed_tiled",

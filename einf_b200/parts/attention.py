@@ -186,6 +186,8 @@ class PagedAttention(Mixer):
         self.out_weight = runtime.matrix(tensors["o_proj.weight"])
         self.out_bias = runtime.vector(tensors["o_proj.bias"]) if spec.get("out_bias", False) else None
         self.position = build_nested("position", spec["position"], tensors, runtime)
+        if getattr(self.position, "amplitude", 1.0) != 1.0:
+            raise ValueError("a rotation with a factor on cosine and sine is taken by the latent mixer's kernels only")
         self.keep_first = int(spec.get("keep_first") or 0)
         if self.keep_first and self.window is None:
             raise ValueError("keep_first needs a window")

@@ -5,7 +5,8 @@ residual stream ``h`` is a 32-bit tensor; a sublayer's output stays *pending*
 until the next norm adds it, so each add is fused with the norm that follows
 (``src/einf/executors/torch/qwen.py:526-563``).  ``prenorm_mixer`` has no feed-forward, ``parallel``
 feeds mixer and feed-forward from one norm, ``prenorm_stream`` adds a residual multiplier,
-convolutions in front of the sublayers, a per-layer token input and a weighted sum over the depth.
+convolutions in front of the sublayers, a per-layer token input and a weighted sum over the depth,
+``prenorm_hyper`` reads and writes several residual streams through vectors and matrices of its own.
 """
 from __future__ import annotations
 
@@ -193,3 +194,45 @@ class PreNormStreamBlock(Block):
             None if depth is None else (history, depth.index, depth.weight),
         )
         return None
+
+
+@register_part("block", "prenorm_hyper")
+class PreNormHyperBlock(Block):
+    """Mixer and feed-forward on several residual streams (:class:`~einf_b200.parts.stream.ResidualStreams`):
+    each sublayer has a connection that says what it reads of the streams, how they mix and what its
+    output adds to each; the feed-forward with its norm and connection is optional.  ``residual`` is the
+    streams; the write of the sublayer that ran last stays pending until the next norm."""
+
+    optional_roles = ("feed_forward_connection", "feed_forward_norm", "feed_forward")
+
+    @classmethod
+    def part_categories(cls):
+        return {
+            "mixer_connection": "stream",
+            "mixer_norm": "norm",
+            "mixer": "mixer",
+            "feed_forward_connection": "stream",
+            "feed_forward_norm": "norm",
+            "feed_forward": "feed_forward",
+        }
+
+    def __init__(self, layer_spec, tensors, runtime):
+        self.runtime = runtime
+        self.spec = layer_spec
+        for role, category in self.part_categories().items():
+            part = None
+            if role in layer_spec.parts:
+                part = build_part(category, layer_spec.parts[role], tensors, runtime)
+            elif role not in self.optional_roles:
+                raise KeyError(f"a prenorm_hyper layer needs the part {role!r}")
+            setattr(self, role, part)
+        if len({part is None for part in (self.feed_forward, self.feed_forward_norm, self.feed_forward_connection)}) > 1:
+            raise ValueError("a feed-forward, its norm and its connection come together")
+
+    def forward(self, residual, pending, ctx, cache):
+        x = residual.normalise(self.mixer_norm, pending, self.mixer_connection)
+        pending = self.mixer.forward(x, ctx, cache)
+        if self.feed_forward is None:
+            return pending
+        x = residual.normalise(self.feed_forward_norm, pending, self.feed_forward_connection)
+        return self.feed_forward.forward(x, ctx)

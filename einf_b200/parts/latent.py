@@ -6,14 +6,20 @@ head ``[dim plain | rot_dim rotated]``; ``W_dkv h`` gives the latent ``c = rms(f
 key part ``r = rotate(last rot_dim)``.  Head h's key is ``[W_uk[h] c | r]``, its value ``W_uv[h] c``; scores
 ``(q_plain . k_plain + q_rot . r) * scale``, causal softmax, then the output projection.
 
+Options, each from the spec: ``q_rank`` None, queries without a latent, ``q = W_q h`` (one product then gives
+everything that h is projected to, and one kernel takes it apart); ``window``, the last that many keys
+only; ``sink``, a stored number per head whose exponential joins the softmax's denominator, with no key and
+no value; ``head_gate``, head h's mixed values are multiplied by ``sigmoid(W_g x)_h`` (in 32-bit, by the
+attention kernel as it divides by the softmax's sum: the value up-projection is linear).
+
 The cache holds the row ``[c | r]`` per token: one key/value head of size ``kv_rank + rot_dim`` whose first
 ``kv_rank`` elements double as the value.  The key up-projection is absorbed into the query
 (``q_plain . W_uk[h] c = (W_uk[h]^T q_plain) . c``) and the value up-projection applied after the
 mixing (``sum_j p_j W_uv[h] c_j = W_uv[h] sum_j p_j c_j``), so attention runs on the cached rows as they
 are, with every query head on the one cached head.
 
-Where a cached row has 64 or 128 elements (bfloat16) the tensor-core attention kernels take it as key
-and as value at once: the mixed rows then carry ``rot_dim`` elements more than the value up-projection
+Where a cached row has 64 or 128 elements (bfloat16; without a query latent a shorter row is filled up
+with zeros) the tensor-core attention kernels take it as key and as value at once: the mixed rows then carry ``rot_dim`` elements more than the value up-projection
 reads (a fifth to a quarter more work in the second product, none in memory traffic).  Other row
 sizes, and the 32-bit path, run the general kernel, which reads the values out of the key rows.
 """
@@ -32,11 +38,21 @@ class LatentAttention(Mixer):
     def tensor_specs(cls, spec):
         hidden, heads = spec["hidden_size"], spec["num_heads"]
         dim, rot, value = spec["head_size"], spec["rotary_size"], spec["value_head_size"]
-        kv_rank, q_rank = spec["kv_rank"], spec["q_rank"]
+        kv_rank, q_rank = spec["kv_rank"], spec.get("q_rank")
+        if q_rank:
+            queries = {
+                "q_down.weight": TensorSpec((q_rank, hidden)),
+                "q_norm.weight": TensorSpec((q_rank,), "scale"),
+                "q_up.weight": TensorSpec((heads * (dim + rot), q_rank)),
+            }
+        else:
+            queries = {"q_proj.weight": TensorSpec((heads * (dim + rot), hidden))}
+        if spec.get("sink"):
+            queries["sink"] = TensorSpec((heads,), "bias")
+        if spec.get("head_gate"):
+            queries["head_gate.weight"] = TensorSpec((heads, hidden))
         return {
-            "q_down.weight": TensorSpec((q_rank, hidden)),
-            "q_norm.weight": TensorSpec((q_rank,), "scale"),
-            "q_up.weight": TensorSpec((heads * (dim + rot), q_rank)),
+            **queries,
             "kv_down.weight": TensorSpec((kv_rank + rot, hidden)),
             "kv_norm.weight": TensorSpec((kv_rank,), "scale"),
             "k_up.weight": TensorSpec((heads * dim, kv_rank)),
@@ -46,10 +62,18 @@ class LatentAttention(Mixer):
 
     @classmethod
     def kernel_libraries(cls, spec, runtime):
-        row = int(spec["kv_rank"]) + int(spec["rotary_size"])
+        row = cls._row_size(spec, runtime.dtype)
         fast = (f"attention_tcgen05:HEAD_SIZE={row}",) if cls._row_on_tensor_cores(row, runtime.dtype) else ()
         return ("pointwise", "latent", "attention_generic", "gemm_simt") + \
             (("gemm_tcgen05",) if runtime.dtype == torch.bfloat16 else ()) + fast
+
+    @staticmethod
+    def _row_size(spec, dtype) -> int:
+        """Elements of a cached row: latent and key part, and zeros up to a size the tensor-core kernels take."""
+        row = int(spec["kv_rank"]) + int(spec["rotary_size"])
+        if not spec.get("q_rank") and dtype == torch.bfloat16 and row <= 128:
+            return 64 if row <= 64 else 128
+        return row
 
     @staticmethod
     def _row_on_tensor_cores(row: int, dtype) -> bool:
@@ -63,10 +87,13 @@ class LatentAttention(Mixer):
         self.rot_dim = int(spec["rotary_size"])
         self.value_size = int(spec["value_head_size"])
         self.kv_rank = int(spec["kv_rank"])
-        self.q_rank = int(spec["q_rank"])
+        self.q_rank = int(spec.get("q_rank") or 0)
         self.scale = float(spec["scale"])
         self.eps = float(spec["eps"])
-        self.row = self.kv_rank + self.rot_dim
+        self.window = spec.get("window")
+        if self.window is not None and self.window <= 0:
+            raise ValueError(f"window must be positive, got {self.window}")
+        self.row = self._row_size(spec, runtime.dtype)
         if self.row > ops.MAX_GENERIC_HEAD_SIZE:
             raise ops.UnsupportedSize(
                 f"latent rows of {self.row} elements: the attention kernel takes up to {ops.MAX_GENERIC_HEAD_SIZE}")
@@ -74,11 +101,24 @@ class LatentAttention(Mixer):
         if 2 * self.position.inv_freq.shape[0] != self.rot_dim:
             raise ValueError("the position encoding must rotate the whole rotated key part")
         heads = self.num_heads
-        # one product for both down-projections: [query latent | kv latent | key part]
-        self.down_weight = runtime.matrix(torch.cat([tensors["q_down.weight"], tensors["kv_down.weight"]], dim=0))
-        self.q_norm = runtime.vector(tensors["q_norm.weight"])
+        self.gated = bool(spec.get("head_gate"))
+        if self.q_rank:
+            if self.gated:
+                raise ValueError("a gate per head comes with queries that have no latent")
+            # one product for both down-projections: [query latent | kv latent | key part]
+            rows = [tensors["q_down.weight"], tensors["kv_down.weight"]]
+            self.q_norm = runtime.vector(tensors["q_norm.weight"])
+            self.q_up = runtime.matrix(tensors["q_up.weight"])
+        else:
+            # one product for everything: [kv latent | key part | queries | gate logits]
+            rows = [tensors["kv_down.weight"], tensors["q_proj.weight"]]
+            if self.gated:
+                rows.append(tensors["head_gate.weight"])
+        if len({m.dtype for m in rows}) > 1:
+            rows = [m.to(torch.float32) for m in rows]
+        self.down_weight = runtime.matrix(torch.cat(rows, dim=0))
         self.kv_norm = runtime.vector(tensors["kv_norm.weight"])
-        self.q_up = runtime.matrix(tensors["q_up.weight"])
+        self.sink = runtime.vector(tensors["sink"]) if spec.get("sink") else None
         # absorbed into the query: per head [kv_rank, dim], the transpose of the key up-projection
         k_up = tensors["k_up.weight"].reshape(heads, self.dim, self.kv_rank)
         self.k_up_t = runtime.matrix(k_up.transpose(1, 2).contiguous())
@@ -91,35 +131,61 @@ class LatentAttention(Mixer):
         singles = int(ctx.single_tokens.shape[0])
         if not singles:
             return ()
+        context = self._visible(ctx.max_context_len)
         if not (self.fast and ops.has_tcgen05_attention(self.row, page_size)):
             # the shared-row decode kernel cuts a token's keys by the batch and the longest context
-            return ("shares", ops.latent_decode_splits(singles, self.num_heads, ctx.max_context_len)) if ctx.decode_only else ()
-        return ops.decode_plan(singles, self.num_heads, 1, self.row, page_size, ctx.max_context_len)
+            return ("shares", ops.latent_decode_splits(singles, self.num_heads, context)) if ctx.decode_only else ()
+        return ops.decode_plan(singles, self.num_heads, 1, self.row, page_size, context)
+
+    def _visible(self, context: int) -> int:
+        return min(context, self.window) if self.window else context
 
     def launch_group(self):
-        return ("latent_attention", self.num_heads, self.row, self.fast)
+        return ("latent_attention", self.num_heads, self.row, self.fast, self.window)
 
     def cache_need(self):
         # the values are the first kv_rank elements of the rows: no value cache of its own
-        return PagedKVNeed(1, self.row, None, 0)
+        return PagedKVNeed(1, self.row, self.window, 0)
+
+    def _queries_and_store(self, x, ctx: StepContext, cache: CacheView):
+        """Project, write the step's cache rows, and return the queries' plain parts ``[T, H, dim]``, the full
+        queries ``[T, H, row]`` with the rotated part in place, and the heads' gates."""
+        tokens, heads, dim = x.shape[0], self.num_heads, self.dim
+        dtype, device = self.runtime.dtype, x.device
+        interleaved = getattr(self.position, "interleaved", False)
+        amplitude = self.position.amplitude
+        writes = cache.writes and cache.k is not None
+        slots, pages = (ctx.slots[cache.group], cache.k) if writes else (None, None)
+        q_full = torch.empty((tokens, heads, self.row), dtype=dtype, device=device)
+        down = ops.project(x, self.down_weight, ctx.status)
+        if not self.q_rank:
+            gate = torch.empty((tokens, heads), dtype=torch.float32, device=device) if self.gated else None
+            first, per_head = self.kv_rank + self.rot_dim, dim + self.rot_dim
+            if down.dim() == 2 and down.dtype == dtype and not any(n % 8 for n in (first, per_head, down.shape[1])):
+                # the plain parts stay where the product left them (16-byte aligned rows)
+                q_plain, copy = down[:, first:first + heads * per_head].unflatten(1, (heads, per_head))[..., :dim], None
+            else:
+                q_plain = copy = torch.empty((tokens, heads, dim), dtype=dtype, device=device)
+            ops.latent_qkv_store(
+                down, self.kv_rank, self.rot_dim, self.kv_norm, self.eps, ctx.positions, self.position.inv_freq,
+                interleaved, amplitude, slots, copy, q_full, gate, pages, ctx.status, dim,
+            )
+            return q_plain, q_full, gate
+        q_latent = torch.empty((tokens, self.q_rank), dtype=dtype, device=device)
+        ops.latent_down_store(
+            down, self.q_rank, self.kv_rank, self.rot_dim, self.q_norm, self.kv_norm, self.eps, ctx.positions,
+            self.position.inv_freq, interleaved, slots, q_latent, pages, ctx.status, amplitude,
+        )
+        q = ops.project(q_latent, self.q_up, ctx.status)
+        q_plain = torch.empty((tokens, heads, dim), dtype=dtype, device=device)
+        ops.latent_q_store(q, ctx.positions, self.position.inv_freq, interleaved, q_plain, q_full, amplitude)
+        return q_plain, q_full, None
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
         tokens = x.shape[0]
         dtype, device = self.runtime.dtype, x.device
         heads = self.num_heads
-        interleaved = getattr(self.position, "interleaved", False)
-        down = ops.project(x, self.down_weight, ctx.status)
-        q_latent = torch.empty((tokens, self.q_rank), dtype=dtype, device=device)
-        writes = cache.writes and cache.k is not None
-        ops.latent_down_store(
-            down, self.q_rank, self.kv_rank, self.rot_dim, self.q_norm, self.kv_norm, self.eps, ctx.positions,
-            self.position.inv_freq, interleaved, ctx.slots[cache.group] if writes else None, q_latent,
-            cache.k if writes else None, ctx.status,
-        )
-        q = ops.project(q_latent, self.q_up, ctx.status)
-        q_plain = torch.empty((tokens, heads, self.dim), dtype=dtype, device=device)
-        q_full = torch.empty((tokens, heads, self.row), dtype=dtype, device=device)
-        ops.latent_q_store(q, ctx.positions, self.position.inv_freq, interleaved, q_plain, q_full)
+        q_plain, q_full, gate = self._queries_and_store(x, ctx, cache)
         ops.per_head_project(q_plain, self.k_up_t, q_full[:, :, : self.kv_rank])
         table = ctx.block_tables[cache.group]
         if self.fast and ops.has_tcgen05_attention(self.row, cache.k.shape[2]):
@@ -127,13 +193,14 @@ class LatentAttention(Mixer):
             mixed_rows = torch.empty((tokens, heads, self.row), dtype=dtype, device=device)
             if ctx.single_tokens.shape[0]:
                 ops.paged_decode_attention_auto(
-                    q_full, cache.k, cache.k, table, ctx.seq_of_token, ctx.positions, mixed_rows, self.scale, None,
-                    ctx.status, None if ctx.decode_only else ctx.single_tokens, max_context=ctx.max_context_len,
+                    q_full, cache.k, cache.k, table, ctx.seq_of_token, ctx.positions, mixed_rows, self.scale,
+                    self.window, ctx.status, None if ctx.decode_only else ctx.single_tokens,
+                    max_context=ctx.max_context_len, sink=self.sink, gate=gate,
                 )
             if ctx.q_tiles.shape[0]:
                 ops.paged_prefill_attention(
-                    q_full, cache.k, cache.k, table, ctx.q_tiles, mixed_rows, self.scale, None, ctx.status,
-                    cached_before=ctx.max_portion_start,
+                    q_full, cache.k, cache.k, table, ctx.q_tiles, mixed_rows, self.scale, self.window, ctx.status,
+                    cached_before=ctx.max_portion_start, sink=self.sink, gate=gate,
                 )
             mixed_latent = mixed_rows[:, :, : self.kv_rank]
         elif ctx.decode_only:
@@ -141,13 +208,14 @@ class LatentAttention(Mixer):
             mixed_latent = torch.empty((tokens, heads, self.kv_rank), dtype=dtype, device=device)
             ops.latent_decode_attention(
                 q_full, cache.k, table, ctx.seq_of_token, ctx.positions, mixed_latent, self.scale,
-                ops.latent_decode_splits(tokens, heads, ctx.max_context_len), ctx.status,
+                ops.latent_decode_splits(tokens, heads, self._visible(ctx.max_context_len)), ctx.status,
+                self.window, self.sink, gate,
             )
         else:
             mixed_latent = torch.empty((tokens, heads, self.kv_rank), dtype=dtype, device=device)
             ops.paged_attention_generic(
                 q_full, cache.k, None, table, ctx.seq_of_token, ctx.positions, mixed_latent,
-                self.scale, None, ctx.status, values_in_keys=self.kv_rank,
+                self.scale, self.window, ctx.status, values_in_keys=self.kv_rank, sink=self.sink, gate=gate,
             )
         mixed = torch.empty((tokens, heads, self.value_size), dtype=dtype, device=device)
         ops.per_head_project(mixed_latent, self.v_up, mixed)

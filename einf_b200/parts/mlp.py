@@ -1,5 +1,5 @@
 """Feed-forwards.  ``gated_mlp``: ``down(act(gate(x)) * up(x))`` with SiLU or the tanh form of GELU; ``dense_mlp``: ``down(act(up(x)))``
-with the square of ReLU (``relu2``), the tanh form of GELU, SiLU or ReLU.
+with the square of ReLU (``relu2``), GELU (the exact form or the tanh form), SiLU or ReLU.
 
 Gate and up share one matrix product on the concatenated weight, gate rows
 first (``src/einf/executors/torch/qwen.py:163-172,206-208``); the activation is

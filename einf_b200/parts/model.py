@@ -17,6 +17,7 @@ from .base import (
     pages_of, state_of, walk_part_specs,
 )
 from .block import build_block
+from .stream import ResidualStreams
 
 
 def _part_specs(model_spec: ModelSpec):
@@ -133,6 +134,8 @@ class DecoderModel:
         """Run the step's tokens through every schedule entry; float logits ``[S, vocab]``
         at ``ctx.logit_rows``."""
         residual = self.embedding.forward(ctx)
+        if self.spec.streams is not None:
+            return self._forward_streams(residual, ctx, caches)
         # the stream is updated in place: entries that take the embedding output again get a copy of it
         first = residual.clone() if any(entry.add_embedding for entry in self.schedule) else None
         pending = None
@@ -149,3 +152,12 @@ class DecoderModel:
         else:
             x = self.final_norm.forward(pending, residual, rows=ctx.logit_rows)
         return self.head.forward(x, ctx.status)
+
+    def _forward_streams(self, first: torch.Tensor, ctx: StepContext, caches: list[CacheView]) -> torch.Tensor:
+        """The same for a model of several residual streams, which its blocks carry along; the head
+        reads the norm of their sum."""
+        streams = ResidualStreams(first, self.spec.streams)
+        pending = None
+        for index, entry in enumerate(self.schedule):
+            pending = self.blocks[entry.layer].forward(streams, pending, ctx, caches[index])
+        return self.head.forward(streams.normalise(self.final_norm, pending, rows=ctx.logit_rows), ctx.status)

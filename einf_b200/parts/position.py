@@ -13,7 +13,12 @@ the general store kernel of the attention mixer rotates that layout.  With ``sca
 ``low``, ``high``, ``original``) a frequency f of wavelength l = 2 pi / f stays as it is where
 l < original / high, becomes f / factor where l > original / low, and between the two is
 ``(1 - s) f / factor + s f`` with ``s = (original / l - low) / (high - low)``: long wavelengths are
-stretched, short ones kept.
+stretched, short ones kept.  ``scaling`` of ``kind: "yarn"`` (``factor``, ``original``, ``fast``, ``slow``) goes by
+the pair's place instead: with ``dim(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta)`` the pair that
+turns t times over the original length, ``lo = max(floor(dim(fast)), 0)`` and ``hi = min(ceil(dim(slow)),
+rotary_dim - 1)``, pair i keeps the share ``1 - r`` of its frequency and has the share r divided by
+``factor``, ``r = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)``; ``amplitude = 0.1 ln(factor) + 1`` then
+multiplies cosine and sine (1 without this scaling; the latent mixer's kernels take it).
 
 ``none``: no encoding; bias and the cache write only.
 """
@@ -67,8 +72,13 @@ class RotaryPosition(PositionEncoding):
             raise ValueError(f"rotary layout must be halves or interleaved, got {self.layout!r}")
         self.interleaved = self.layout == "interleaved"
         scaling = spec.get("scaling")
+        #: factor on cosine and sine
+        self.amplitude = 1.0
         if scaling is None:
             inv_freq = 1.0 / (self.theta ** (torch.arange(0, self.rotary_dim, 2).float() / self.rotary_dim))
+        elif scaling.get("kind") == "yarn":
+            inv_freq = self.yarn_frequencies(self.theta, self.rotary_dim, scaling)
+            self.amplitude = 0.1 * math.log(float(scaling["factor"])) + 1.0
         else:
             inv_freq = self.scaled_frequencies(self.theta, self.rotary_dim, scaling)
         self.inv_freq = inv_freq.to(runtime.device)
@@ -89,9 +99,27 @@ class RotaryPosition(PositionEncoding):
             table.append(f)
         return torch.tensor(table, dtype=torch.float64).to(torch.float32)
 
+    @staticmethod
+    def yarn_frequencies(theta: float, rotary_dim: int, scaling) -> torch.Tensor:
+        """The frequency table with a ramp over the pairs, made in 64-bit on the host."""
+        factor, original, fast, slow = (float(scaling[k]) for k in ("factor", "original", "fast", "slow"))
+
+        def dim_of(turns: float) -> float:
+            return rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+
+        low, high = max(math.floor(dim_of(fast)), 0), min(math.ceil(dim_of(slow)), rotary_dim - 1)
+        table = []
+        for i in range(rotary_dim // 2):
+            f = theta ** (-2.0 * i / rotary_dim)
+            ramp = min(max((i - low) / max(high - low, 0.001), 0.0), 1.0)
+            table.append(f / factor * ramp + f * (1.0 - ramp))
+        return torch.tensor(table, dtype=torch.float64).to(torch.float32)
+
     def encode_and_store(self, qkv, bias, ctx, cache, q_out, num_heads, num_kv_heads, head_size):
         if self.rotary_dim > head_size:
             raise ValueError(f"rotary_dim {self.rotary_dim} exceeds head size {head_size}")
+        if self.amplitude != 1.0:
+            raise ValueError("a factor on cosine and sine is taken by the latent mixer's kernels only")
         if self.interleaved:
             raise ValueError("the interleaved layout is rotated by the attention mixer's general store kernel")
         _store(self.inv_freq, qkv, bias, ctx, cache, q_out, num_heads, num_kv_heads, head_size)
@@ -106,6 +134,7 @@ class NoPosition(PositionEncoding):
     def __init__(self, spec, tensors, runtime):
         super().__init__(spec, tensors, runtime)
         self.inv_freq = torch.empty(0, dtype=torch.float32, device=runtime.device)
+        self.amplitude = 1.0
 
     def encode_and_store(self, qkv, bias, ctx, cache, q_out, num_heads, num_kv_heads, head_size):
         _store(self.inv_freq, qkv, bias, ctx, cache, q_out, num_heads, num_kv_heads, head_size)

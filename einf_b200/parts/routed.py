@@ -2,14 +2,15 @@
 
 ``routed_mlp``: router logits ``z = W_router x`` in 32-bit; the ``top_k`` experts with the largest
 scores (``score``: ``sigmoid`` or ``softmax`` over all experts; ``renormalise`` divides the chosen
-weights by their sum); an expert is ``down(silu(gate(u)) * up(u))`` without biases.  With
+weights by their sum, to which ``renormalise_eps`` is added; ``weight_scale`` multiplies the weights);
+an expert is ``down(silu(gate(u)) * up(u))`` without biases.  With
 ``weight_on: "input"`` the expert sees ``u = w x`` and its output is added as it is; with ``"output"``
 it sees x and its output is multiplied by w.
 
 Optional, each from the spec.  ``correction``: a stored number per router output that is added to the
 scores for the choice alone (the weights stay the scores).  ``groups`` (``count``, ``keep``): the router's
 outputs form equal groups of neighbours, and only those of the ``keep`` groups whose best choice score
-is largest can be chosen.  ``num_identity``: the router has that many outputs beyond the experts;
+is largest can be chosen (with ``best`` 2 in the groups: whose two best together are largest).  ``num_identity``: the router has that many outputs beyond the experts;
 one of those, when chosen, hands the token through unchanged (times its weight) and has no tensors.
 They count in the softmax, in the groups and in ``top_k`` like any expert.  ``shared`` (an
 ``intermediate_size``): one more gated feed-forward that every token takes, added to the sum; with
@@ -69,6 +70,8 @@ class RoutedMLP(FeedForward):
         if self.score not in ops.ROUTER_SCORES:
             raise ValueError(f"router score must be one of {sorted(ops.ROUTER_SCORES)}, got {self.score!r}")
         self.renormalise = bool(spec.get("renormalise", False))
+        self.renormalise_eps = float(spec.get("renormalise_eps") or 0.0)
+        self.weight_scale = float(spec.get("weight_scale", 1.0))
         weight_on = str(spec.get("weight_on", "output"))
         if weight_on not in ("input", "output"):
             raise ValueError(f"weight_on must be input or output, got {weight_on!r}")
@@ -79,10 +82,13 @@ class RoutedMLP(FeedForward):
             raise ValueError(f"top_k {self.top_k} of {self.num_outputs} router outputs")
         if self.num_identity and self.weight_on_input:
             raise ValueError("experts that hand their input through take their weight on the output")
-        self.groups = None
+        self.groups, self.group_best = None, 1
         if spec.get("groups"):
             self.groups = (int(spec["groups"]["count"]), int(spec["groups"]["keep"]))
             count, keep = self.groups
+            self.group_best = int(spec["groups"].get("best", 1))
+            if self.group_best not in (1, 2):
+                raise ValueError(f"a group is scored by its best one or two outputs, not {self.group_best}")
             if count <= 0 or self.num_outputs % count or not 0 < keep <= count or \
                     self.top_k > keep * (self.num_outputs // count):
                 raise ValueError(f"{self.num_outputs} router outputs in {count} groups of which {keep} are kept "
@@ -116,7 +122,8 @@ class RoutedMLP(FeedForward):
         expert_ids = torch.empty((tokens, top_k), dtype=torch.int32, device=device)
         weights = torch.empty((tokens, top_k), dtype=torch.float32, device=device)
         ops.router_topk(logits, top_k, self.score, self.renormalise, expert_ids, weights, self.num_outputs,
-                        self.correction, self.groups)
+                        self.correction, self.groups, group_best=self.group_best,
+                        renormalise_eps=self.renormalise_eps, weight_scale=self.weight_scale)
         addend_gate = None
         if self.shared_size:
             if add is not None:

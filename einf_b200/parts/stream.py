@@ -15,6 +15,12 @@ layer i is ``sum_(j <= i + 1) w[j] X_j``.  The results of all layers of the step
 
 The parts hold tensors and sizes; the block that arranges them (``prenorm_stream``) launches one
 kernel for the end of a layer: pending sublayer output, token input and weighted sum together.
+
+``hyper_connection``: the model has several residual streams x_1 .. x_s instead of one
+(:class:`ResidualStreams`), all equal to the embedding output at the start.  A sublayer reads ``u = sum_s
+read[s] x_s`` and, with y its output, every stream becomes ``x_t <- sum_s mix[s, t] x_s + write[t] y``.  The
+write of one sublayer, what the next one reads and its norm are one launch (``ops.hyper_norm``), so
+between sublayers y stays pending as it does for a single stream.
 """
 from __future__ import annotations
 
@@ -105,3 +111,71 @@ class DepthAverage(Part):
         if history is None or history.shape[1:] != residual.shape:
             raise RuntimeError("a depth average runs before the first layer of the step has made the history")
         return history
+
+
+@register_part("stream", "hyper_connection")
+class HyperConnection(Part):
+    @classmethod
+    def tensor_specs(cls, spec):
+        streams = spec["streams"]
+        return {
+            "read": TensorSpec((streams,), "mean"),
+            "write": TensorSpec((streams,), "scale"),
+            "mix": TensorSpec((streams, streams), "near_identity"),
+        }
+
+    @classmethod
+    def kernel_libraries(cls, spec, runtime):
+        return ("hyper",)
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.streams = int(spec["streams"])
+        if not 1 <= self.streams <= ops.MAX_STREAMS:
+            raise ops.UnsupportedSize(f"{self.streams} residual streams: the kernel takes 1 to {ops.MAX_STREAMS}")
+        self.read = runtime.vector(tensors["read"])
+        self.write = runtime.vector(tensors["write"])
+        self.mix = runtime.vector(tensors["mix"])       # [from, to]
+
+
+class ResidualStreams:
+    """The residual streams of a step, in the place of the one residual tensor: 32-bit ``[streams, T,
+    hidden]``, or the one tensor ``[T, hidden]`` they all still equal before the first write.  The
+    connection of the sublayer that ran last stays with them until its output, pending, is written."""
+
+    def __init__(self, first: torch.Tensor, count: int) -> None:
+        self.values, self.count = first, count
+        self.connection: HyperConnection | None = None
+
+    def normalise(self, norm, pending, connection=None, rows=None) -> torch.Tensor:
+        """Write what is pending, and return the norm of what ``connection``'s sublayer reads (without
+        one: of the sum of the streams) at all rows, or at ``rows``, for which nothing is stored."""
+        before = self.connection
+        if (pending is None) != (before is None):
+            raise ValueError("a sublayer's output and its connection are written together")
+        values = self.values
+        tokens, hidden = values.shape[-2:]
+        target = None
+        if before is not None and rows is None:
+            target = values if values.dim() == 3 else torch.empty((self.count, tokens, hidden), dtype=torch.float32,
+                                                                  device=values.device)
+        out = torch.empty((tokens if rows is None else rows.shape[0], hidden), dtype=norm.runtime.dtype,
+                          device=values.device)
+        ops.hyper_norm(
+            pending, values, self.count, None if before is None else (before.mix, before.write),
+            None if connection is None else connection.read, target, norm.weight, norm.bias, norm.centre, norm.eps,
+            out, rows,
+        )
+        if target is not None:
+            self.values = target
+        self.connection = connection
+        return out
+
+    def total(self, pending) -> torch.Tensor:
+        """The sum of the streams with what is pending written, ``[T, hidden]`` (for a look at the model
+        from outside; the step itself never needs it)."""
+        values = self.values if self.values.dim() == 3 else self.values.expand(self.count, *self.values.shape)
+        if pending is None:
+            return values.sum(0)
+        y = (pending.sum(0) if pending.dim() == 3 else pending).float()
+        return (self.connection.mix.sum(1)[:, None, None] * values).sum(0) + self.connection.write.sum() * y

@@ -97,7 +97,7 @@ def project(x, weight, status, out_dtype=None, allow_partial=True):
 
 
 def paged_attention_generic(q, k_cache, v_cache, block_table, seq_of_token, positions, out, scale, window, status,
-                            chunk=None, softcap=None, keep_first=0, values_in_keys=None, sink=None):
+                            chunk=None, softcap=None, keep_first=0, values_in_keys=None, sink=None, gate=None):
     tokens, num_heads, head_size = q.shape
     _, num_kv_heads, page_size, _ = k_cache.shape
     groups = num_heads // num_kv_heads
@@ -122,12 +122,14 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, seq_of_token, posi
         if sink is not None:        # one more column in the denominator, with no value
             scores = torch.cat([scores, sink.float()[:, None]], dim=1)
         probabilities = torch.softmax(scores, dim=-1)[:, :keys.shape[0]]
-        out[t] = torch.einsum("hn,nhd->hd", probabilities, v).to(out.dtype)
+        mixed = torch.einsum("hn,nhd->hd", probabilities, v)
+        out[t] = (mixed if gate is None else gate[t][:, None] * mixed).to(out.dtype)
 
 
-def latent_decode_attention(q, cache, block_table, seq_of_token, positions, out, scale, splits, status):
-    paged_attention_generic(q, cache, None, block_table, seq_of_token, positions, out, scale, None, status,
-                            values_in_keys=out.shape[2])
+def latent_decode_attention(q, cache, block_table, seq_of_token, positions, out, scale, splits, status, window=None,
+                            sink=None, gate=None):
+    paged_attention_generic(q, cache, None, block_table, seq_of_token, positions, out, scale, window, status,
+                            values_in_keys=out.shape[2], sink=sink, gate=gate)
 
 
 def latent_decode_splits(num_tokens, num_heads, max_context):
@@ -149,6 +151,8 @@ def activation(x, out, kind):
         y = z / (1 + torch.exp(-z))
     elif kind == "relu":
         y = torch.clamp(z, min=0)
+    elif kind == "gelu":
+        y = 0.5 * z * (1 + torch.erf(z * 2.0 ** -0.5))
     else:
         raise ValueError(kind)
     out.copy_(y.to(out.dtype))
@@ -220,14 +224,14 @@ def qkv_norm_store(qkv, bias, slots, q_out, k_cache, v_cache, num_heads, num_kv_
 
 
 def latent_down_store(down, q_rank, kv_rank, rot_dim, q_norm_weight, kv_norm_weight, eps, positions, inv_freq,
-                      interleaved, slots, q_latent_out, cache, status):
+                      interleaved, slots, q_latent_out, cache, status, amplitude=1.0):
     values = _summed(down)
     q_latent, latent, part = values.split([q_rank, kv_rank, rot_dim], dim=-1)
     if q_rank:
         q_latent = q_latent * torch.rsqrt(q_latent.pow(2).mean(-1, keepdim=True) + eps) * q_norm_weight
         q_latent_out.copy_(q_latent.to(q_latent_out.dtype))
     latent = latent * torch.rsqrt(latent.pow(2).mean(-1, keepdim=True) + eps) * kv_norm_weight
-    part = _rotate(part[:, None, :], positions, inv_freq, interleaved)[:, 0]
+    part = amplitude * _rotate(part[:, None, :], positions, inv_freq, interleaved)[:, 0]
     if slots is not None:
         page_size = cache.shape[2]
         keep = slots >= 0
@@ -236,12 +240,58 @@ def latent_down_store(down, q_rank, kv_rank, rot_dim, q_norm_weight, kv_norm_wei
         cache[page, 0, offset, :] = torch.cat([latent, part], dim=-1)[keep].to(cache.dtype)
 
 
-def latent_q_store(q, positions, inv_freq, interleaved, q_plain, q_full):
+def latent_q_store(q, positions, inv_freq, interleaved, q_plain, q_full, amplitude=1.0):
     tokens, heads, dim = q_plain.shape
     rot_dim = 2 * inv_freq.shape[0]
     values = _summed(q).reshape(tokens, heads, dim + rot_dim)
     q_plain.copy_(values[..., :dim].to(q_plain.dtype))
-    q_full[..., q_full.shape[2] - rot_dim:] = _rotate(values[..., dim:], positions, inv_freq, interleaved).to(q_full.dtype)
+    q_full[..., q_full.shape[2] - rot_dim:] = (
+        amplitude * _rotate(values[..., dim:], positions, inv_freq, interleaved)).to(q_full.dtype)
+
+
+def latent_qkv_store(product, kv_rank, rot_dim, kv_norm_weight, eps, positions, inv_freq, interleaved, amplitude, slots,
+                     q_plain, q_full, gate, cache, status, dim):
+    tokens, heads, row = q_full.shape
+    values = _summed(product)
+    latent, part, q, logits = values.split([kv_rank, rot_dim, heads * (dim + rot_dim),
+                                            heads if gate is not None else 0], dim=-1)
+    latent = latent * torch.rsqrt(latent.pow(2).mean(-1, keepdim=True) + eps) * kv_norm_weight
+    part = amplitude * _rotate(part[:, None, :], positions, inv_freq, interleaved)[:, 0]
+    if slots is not None:
+        page_size = cache.shape[2]
+        keep = slots >= 0
+        page, offset = (slots[keep] // page_size).long(), (slots[keep] % page_size).long()
+        zeros = torch.zeros((tokens, row - kv_rank - rot_dim), dtype=torch.float32, device=values.device)
+        cache[page, 0, offset, :] = torch.cat([latent, part, zeros], dim=-1)[keep].to(cache.dtype)
+    q = q.reshape(tokens, heads, dim + rot_dim)
+    if q_plain is not None:
+        q_plain.copy_(q[..., :dim].to(q_plain.dtype))
+    q_full[..., kv_rank:] = 0
+    q_full[..., kv_rank:kv_rank + rot_dim] = (
+        amplitude * _rotate(q[..., dim:], positions, inv_freq, interleaved)).to(q_full.dtype)
+    if gate is not None:
+        gate.copy_(torch.sigmoid(logits))
+
+
+def hyper_norm(pending, source, streams, connection, read, dest, weight, bias, centre, eps, out, rows=None):
+    x = source if source.dim() == 3 else source[None].expand(streams, *source.shape)
+    y = None if pending is None else _summed(pending)
+    if connection is not None:
+        mix, write = connection
+        x = torch.einsum("sr,stw->rtw", mix, x)
+        if y is not None:
+            x = x + write[:, None, None] * y
+    elif y is not None:
+        x = x + y
+    if dest is not None:
+        dest.copy_(x.reshape(dest.shape))
+    u = x.sum(0) if read is None else torch.einsum("s,stw->tw", read, x)
+    if rows is not None:
+        u = u[rows.long()]
+    if centre:
+        u = u - u.mean(-1, keepdim=True)
+    u = u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * weight
+    out.copy_((u if bias is None else u + bias).to(out.dtype))
 
 
 def per_head_project(x, weight, out):
@@ -249,7 +299,7 @@ def per_head_project(x, weight, out):
 
 
 def router_topk(logits, top_k, score, renormalise, expert_ids, weights, num_experts=None, correction=None,
-                groups=None):
+                groups=None, group_best=1, renormalise_eps=0.0, weight_scale=1.0):
     z = _summed(logits)
     if num_experts is not None:
         z = z[:, :num_experts]
@@ -259,7 +309,11 @@ def router_topk(logits, top_k, score, renormalise, expert_ids, weights, num_expe
     if groups is not None:
         count, keep = groups
         tokens, experts = choice.shape
-        best = choice.reshape(tokens, count, experts // count).max(dim=-1).values
+        members = choice.reshape(tokens, count, experts // count)
+        best = members.max(dim=-1).values
+        if group_best == 2:         # the sum of a group's two best scores
+            members = scores.reshape(members.shape) if correction is None else members
+            best = torch.sort(members, dim=-1, descending=True).values[..., :2].sum(-1)
         kept = torch.sort(best, dim=-1, descending=True, stable=True).indices[:, :keep]
         allowed = torch.zeros(tokens, count, dtype=torch.bool, device=z.device)
         allowed.scatter_(1, kept, True)
@@ -268,7 +322,8 @@ def router_topk(logits, top_k, score, renormalise, expert_ids, weights, num_expe
     order = torch.sort(choice, dim=-1, descending=True, stable=True).indices[:, :top_k]
     chosen = torch.gather(scores, 1, order)
     if renormalise:
-        chosen = chosen / chosen.sum(-1, keepdim=True)
+        chosen = chosen / (chosen.sum(-1, keepdim=True) + renormalise_eps)
+    chosen = chosen * weight_scale
     expert_ids.copy_(order.to(expert_ids.dtype))
     weights.copy_(chosen)
 
@@ -649,7 +704,7 @@ _NAMES = (
     "gated_norm", "recurrence_plan", "latent_down_store", "latent_q_store", "per_head_project", "router_topk",
     "moe_dispatch", "moe_gemm", "moe_combine", "softcap", "latent_decode_attention", "latent_decode_splits", "moe_gemm_on_tensor_cores", "moe_gemm_splits",
     "act_mul", "norm_conv", "stream_tail", "paged_attention_mixed", "gated_scan", "memory_gates", "memory_output",
-    "norm_join", "memory_value_columns", "recurrence_step_splits",
+    "norm_join", "memory_value_columns", "recurrence_step_splits", "latent_qkv_store", "hyper_norm",
 )
 
 
