@@ -545,18 +545,18 @@ def test_a_far_key_counts_emulated(tmp_path, emulated):
 
 
 def sink_check(tmp_path, dtype, device, rank=24):
-    """A sink as large as the best score takes a good part of every row's weight: left out, counted twice or
-    scaled like a score, it shows."""
+    """A sink as large as the scores takes a good part of most rows' weight: left out, counted twice or scaled
+    like a score, it shows."""
     from einf_b200.engine.replay import TraceReplayer
 
-    config, weights = needle_model(SINK, 9, scale=0.5, sink=3.0, rank=rank)
-    _, without = needle_model(SINK, 9, scale=0.5, sink=-40.0, rank=rank)
+    config, weights = needle_model(SINK, 9, scale=0.2, sink=3.0, rank=rank)
+    _, without = needle_model(SINK, 9, scale=0.2, sink=-40.0, rank=rank)
     folder = tmp_path / "sink"
     write_folder(folder, config, 0, weights)
     requests = {"s": [2 + (i * 5) % 37 for i in range(40)]}
     expected, _ = expected_rows(config, weights, requests)
     other, _ = expected_rows(config, without, requests)
-    assert min(np.abs(expected[key] - other[key]).max() for key in expected) > 0.05
+    assert float(np.quantile([np.abs(expected[key] - other[key]).max() for key in expected], 0.25)) > 0.05
     for steps in (trace_tools.whole(requests), trace_tools.last_one_by_one(requests, tail=20),
                   trace_tools.in_portions(requests, sizes=(5, 2, 9))):
         replayer = TraceReplayer(folder, dtype, 64, block_len=16, device=device)
