@@ -1456,6 +1456,252 @@ def rekodra_kernels(peak: dict) -> dict:
     return out
 
 
+def sorizen_sizes(width: int, heads: int, size: int, ff: int, kv_rank: int, rot_dim: int, vocab: int, window: int,
+                  layers: int) -> dict:
+    """A Sorizen configuration at the layer sizes of a Qwen2 model: the two mixers in turn, dense and
+    routed feed-forwards in turn by pairs (the two of eight experts that a token takes are together as
+    wide as a dense gated feed-forward, the dense one has as many weights), two residual streams."""
+    def mixer(base, factor):
+        return {"heads": heads, "dim": size, "rot_dim": rot_dim, "vdim": size, "kv_rank": kv_rank,
+                "scale": (size + rot_dim) ** -0.5, "mask": {"size": window},
+                "rot": {"base": base, "dims": rot_dim,
+                        "scaling": {"factor": factor, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+
+    dense = {"kind": "dense", "ff": ff * 3 // 2}
+    moe = {"kind": "moe", "expert": {"ff": ff // 2},
+           "router": {"experts": 8, "top": 2, "groups": {"count": 2, "keep": 1}, "scale": 2.5}}
+    made = [{"type": ("latent_attention", "latent_attention_2")[index % 2], "mixer": mixer((1e6, 1e4)[index % 2], 8.0),
+             "mlp": (dense, moe)[index // 2 % 2]} for index in range(layers)]
+    return {"architecture": "Sorizen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": width ** 0.5}, "streams": 2, "layers": made}
+
+
+def run_sorizen(args) -> dict:
+    """Prefill and decode throughput of the Sorizen design at the layer sizes of the 0.5B and 1.5B models
+    (random weights, eight layers unless --layers says otherwise), beside Bomipel, the closest of the
+    other designs (latent attention, routed feed-forwards), and Qwen2, each with as many layers at the
+    same width, heads and vocabulary; then the design's own kernels alone, each beside its like."""
+    import torch
+
+    from einf_b200.cache import CacheManager
+    from einf_b200.config import EngineConfig, config_from_dict
+    from einf_b200.engine import ModelRunner
+    from einf_b200.sampling import Sampler
+
+    layers = args.layers or 8
+    result = {"scenario": "sorizen", "layers": layers, "context": CONTEXT, "window": 1024, "streams": 2}
+    # name: width, dense ff, heads, kv heads, head size, latent rank, rotated part, Bomipel's query rank
+    shapes = {"0.5b": (896, 4864, 14, 2, 64, 96, 32, 384), "1.5b": (1536, 8960, 12, 2, 128, 96, 32, 768),
+              "1.5b-row576": (1536, 8960, 12, 2, 128, 512, 64, 768)}
+    if args.only != "all":          # one small workload for a launch list
+        shapes = {"0.5b": shapes["0.5b"]}
+    for name, (width, ff, heads, kv_heads, size, rank, rot, q_rank) in shapes.items():
+        qwen = dict(SIZES["1.5b"] if name.startswith("1.5b") else QWEN25_05B, num_hidden_layers=layers, tie_word_embeddings=True)
+        vocab = qwen["vocab_size"]
+        ours = sorizen_sizes(width, heads, size, ff, rank, rot, vocab, 1024, layers)
+        near = bomipel_sizes(width, heads, kv_heads, size, ff, 8, 2, rank, rot, q_rank, layers, vocab, 1024, 4)
+        for arch, cfg in (("sorizen", ours), ("bomipel", near), ("qwen2", qwen)):
+            if arch != "sorizen" and (args.only != "all" or (arch == "qwen2" and rank == 512)):
+                continue
+            pages = 64 * (CONTEXT // PAGE + 2) + 64
+            runner = ModelRunner.from_random(
+                config_from_dict(cfg), 0,
+                EngineConfig(dtype="bfloat16", block_len=PAGE, num_blocks=pages, max_batch_len=8192,
+                             max_prefill_chunk_len=8192, max_requests=64, use_cuda_graphs=not args.no_graphs))
+            manager = CacheManager(runner.group_specs(), runner.num_state_slots)
+            sampler = Sampler(runner.runtime.device, 64)
+            prompts = {"decode": (), "prefill": (2048,)}.get(args.only, (2048, 8192))
+            if arch == "bomipel" and rank == 512:
+                prompts = prompts[:1]       # its latent layers see all keys, on the general kernel
+            for tokens in prompts:
+                timed = time_prefill(runner, sampler, manager, tokens, repeats=2 if args.only == "prefill" else 5)
+                result[f"{name}_{arch}_prefill{tokens}_ms"] = round(timed["ms"], 3)
+                result[f"{name}_{arch}_prefill{tokens}_tokens_per_s"] = round(tokens / (timed["ms"] * 1e-3))
+            for batch in {"decode": (args.batch,), "prefill": ()}.get(args.only, (1, 8, 64)):
+                timed = time_decode(runner, sampler, manager, batch, CONTEXT, args.steps, args.warmup,
+                                    min_seconds=0.0 if args.only == "decode" else 0.2)
+                result[f"{name}_{arch}_decode_b{batch}_ms"] = round(timed["ms_per_step"], 3)
+                result[f"{name}_{arch}_decode_b{batch}_tokens_per_s"] = round(timed["tokens_per_s"], 1)
+                result[f"{name}_{arch}_decode_b{batch}_launches_per_step"] = timed["launches"] // max(1, args.steps)
+            del runner, manager, sampler
+            torch.cuda.empty_cache()
+    if args.only not in ("decode", "prefill"):
+        result["kernels"] = sorizen_kernels(peaks())
+    return result
+
+
+def sorizen_kernels(peak: dict) -> dict:
+    """The design's kernels alone (microseconds per launch in a CUDA graph of launches on rotating
+    buffers larger than the L2) with the bytes or flops each must move, each beside the like kernel of
+    another path: the streams' write, read and norm beside the residual norm, the store kernel beside
+    Bomipel's two, windowed latent attention with sink and gate beside the same without."""
+    import torch
+
+    from einf_b200 import ops
+
+    device = torch.device("cuda:0")
+    status = torch.zeros(1, dtype=torch.int32, device=device)
+    out: dict = {}
+    gbs, tflops = peak["hbm_gbs"], peak["bf16_tflops"]
+    turn = [0]
+
+    def rate(key, us, nbytes=0, flops=0):
+        out[key + "_us"] = round(us, 1)
+        if nbytes:
+            out[key + "_hbm_frac"] = round(nbytes / us / 1e3 / gbs, 3)
+        if flops:
+            out[key + "_flops_frac"] = round(flops / us / 1e6 / tflops, 4)
+
+    ops.ensure_built(["routed", "pointwise", "latent", "hyper", "attention_generic", "gemm_tcgen05",
+                      *ops.attention_libraries(128, PAGE)])
+
+    def rotating(make, bytes_each):
+        return [make() for _ in range(max(2, int(300e6 / bytes_each)))]
+
+    def timed(key, fn, buffers, launches=8, nbytes=0, flops=0):
+        def call():
+            turn[0] += 1
+            fn(buffers[turn[0] % len(buffers)])
+
+        rate(key, _graph_time_us(call, max(launches, min(len(buffers), 64))), nbytes, flops)
+
+    for name, width, heads, dim in (("0.5b", 896, 14, 64), ("1.5b", 1536, 12, 128)):
+        weight, bias = torch.ones(width, device=device), torch.zeros(width, device=device)
+        for streams in (2, 4):
+            mix, write, read = torch.randn(streams, streams, device=device), torch.ones(streams, device=device), \
+                torch.ones(streams, device=device)
+            for tokens, splits in ((2048, 1), (8, 12), (64, 12)):
+                def make():
+                    y = torch.randn(splits, tokens, width, device=device) if splits > 1 else \
+                        torch.randn(tokens, width, device=device).bfloat16()
+                    return y, torch.randn(streams, tokens, width, device=device), \
+                        torch.empty(tokens, width, device=device).bfloat16()
+
+                y_bytes = tokens * width * (4 * splits if splits > 1 else 2)
+                nbytes = y_bytes + tokens * width * (8 * streams + 2)
+                timed(f"{name}_t{tokens}_hyper_norm_s{streams}",
+                      lambda b: ops.hyper_norm(b[0], b[1], streams, (mix, write), read, b[1], weight, bias, True, 1e-6, b[2]),
+                      rotating(make, nbytes), nbytes=nbytes)
+                if streams == 2:
+                    timed(f"{name}_t{tokens}_residual_norm",
+                          lambda b: ops.add_rmsnorm(b[0], b[1][0], weight, 1e-6, b[2], None, status),
+                          rotating(make, nbytes), nbytes=y_bytes + tokens * width * 10)
+        for rank, rot in ((96, 32), (512, 64)):
+            row, tag = rank + rot, f"{name}_row{rank + rot}"
+            inv_freq = torch.rand(rot // 2, device=device)
+            norm = torch.ones(rank, device=device)
+            for tokens, splits in ((2048, 1), (8, 6), (64, 6)):
+                product_width = rank + rot + heads * (dim + rot) + heads
+                positions = torch.arange(tokens, dtype=torch.int32, device=device)
+                slots = torch.arange(tokens, dtype=torch.int32, device=device)
+                cache = torch.zeros(tokens // PAGE + 2, 1, PAGE, row, device=device).bfloat16()
+                gate = torch.empty(tokens, heads, device=device)
+
+                def make_product():
+                    shape = (splits, tokens, product_width) if splits > 1 else (tokens, product_width)
+                    product = torch.randn(shape, device=device)
+                    return (product if splits > 1 else product.bfloat16(),
+                            torch.empty(tokens, heads, dim, device=device).bfloat16(),
+                            torch.empty(tokens, heads, row, device=device).bfloat16())
+
+                nbytes = tokens * product_width * (4 * splits if splits > 1 else 2) + tokens * (row + heads * (dim + rot)) * 2
+                timed(f"{tag}_t{tokens}_latent_qkv_store",
+                      lambda b: ops.latent_qkv_store(b[0], rank, rot, norm, 1e-6, positions, inv_freq, True, 1.2, slots, b[1],
+                                                     b[2], gate, cache, status, dim),
+                      rotating(make_product, nbytes), nbytes=nbytes)
+
+                def two(b):
+                    ops.latent_down_store(b[4], 0, rank, rot, None, norm, 1e-6, positions, inv_freq, True, slots, None, cache,
+                                          status)
+                    ops.latent_q_store(b[3], positions, inv_freq, True, b[1], b[2])
+
+                def make_two():
+                    lead = (splits, tokens) if splits > 1 else (tokens,)
+                    q, down = torch.randn(*lead, heads * (dim + rot), device=device), torch.randn(*lead, row, device=device)
+                    if splits == 1:
+                        q, down = q.bfloat16(), down.bfloat16()
+                    return (*make_product(), q, down)
+
+                timed(f"{tag}_t{tokens}_two_stores", two, rotating(make_two, nbytes), nbytes=nbytes)
+        latent_attention_points(name, heads, rate, status, out)
+    for experts, top, groups in ((8, 2, (2, 1)), (64, 6, (8, 3))):
+        for tokens in (8, 2048):
+            logits = torch.randn(tokens, experts, device=device)
+            ids = torch.empty(tokens, top, dtype=torch.int32, device=device)
+            weights = torch.empty(tokens, top, device=device)
+            rate(f"router_e{experts}_t{tokens}_two_best", _graph_time_us(lambda: ops.router_topk(
+                logits, top, "sigmoid", True, ids, weights, experts, None, groups, group_best=2, renormalise_eps=1e-20,
+                weight_scale=2.5), 8))
+            rate(f"router_e{experts}_t{tokens}_best", _graph_time_us(lambda: ops.router_topk(
+                logits, top, "sigmoid", True, ids, weights, experts, None, groups), 8))
+    out["status"] = int(status)
+    return out
+
+
+def latent_attention_points(name: str, heads: int, rate, status, out: dict) -> None:
+    """Attention over rows that are keys and values at once: a prompt of 2,048 and single tokens at 4,096, a
+    window of 1,024 with a sink and a gate beside the same without them and beside all keys."""
+    import torch
+
+    from einf_b200 import ops
+
+    device = status.device
+    window, tokens = 1024, 2048
+    sink = torch.zeros(heads, device=device)
+    for rank, rot in ((96, 32), (128, 16), (512, 64)):
+        row, tag = rank + rot, f"{name}_row{rank + rot}"
+        on_tensor_cores = row in (64, 128)
+        pages = tokens // PAGE
+        tiles = torch.tensor([[0, first, 128, first] for first in range(0, tokens, 128)], dtype=torch.int32, device=device)
+        seq = torch.zeros(tokens, dtype=torch.int32, device=device)
+        pos = torch.arange(tokens, dtype=torch.int32, device=device)
+        table = torch.arange(pages, dtype=torch.int32, device=device).view(1, -1)
+        k = torch.randn(pages + 2, 1, PAGE, row, device=device).bfloat16()
+        q = torch.randn(tokens, heads, row, device=device).bfloat16()
+        gate = torch.rand(tokens, heads, device=device)
+        o = torch.empty(tokens, heads, row if on_tensor_cores else rank, device=device).bfloat16()
+        window_pairs, all_pairs = tokens * window - window * window / 2, tokens * tokens / 2
+        for what, w, s, g, pairs in (("window", window, None, None, window_pairs), ("all", None, None, None, all_pairs),
+                                     ("window_sink_gate", window, sink, gate, window_pairs)):
+            if on_tensor_cores:
+                def run():
+                    ops.paged_prefill_attention(q, k, k, table, tiles, o, row ** -0.5, w, status, cached_before=0, sink=s, gate=g)
+            else:
+                def run():
+                    ops.paged_attention_generic(q, k, None, table, seq, pos, o, row ** -0.5, w, status, values_in_keys=rank,
+                                                sink=s, gate=g)
+            if what == "all" and not on_tensor_cores:
+                continue
+            rate(f"{tag}_prefill{tokens}_{what}", _graph_time_us(run, 4), flops=2 * heads * (row + rank) * pairs)
+        for batch in (8, 64):
+            pages = CONTEXT // PAGE
+            launches = 8
+            seq = torch.arange(batch, dtype=torch.int32, device=device)
+            pos = torch.full((batch,), CONTEXT - 1, dtype=torch.int32, device=device)
+            tables = [torch.arange(i * pages * batch, (i + 1) * pages * batch, dtype=torch.int32, device=device).view(batch, pages)
+                      for i in range(launches)]
+            k = torch.zeros(pages * batch * launches + 2, 1, PAGE, row, device=device, dtype=torch.bfloat16).normal_()
+            q = torch.randn(batch, heads, row, device=device).bfloat16()
+            gate = torch.rand(batch, heads, device=device)
+            o = torch.empty(batch, heads, row if on_tensor_cores else rank, device=device).bfloat16()
+            turn = [0]
+            for what, w, s, g in (("window", window, None, None), ("all", None, None, None),
+                                  ("window_sink_gate", window, sink, gate)):
+                splits = ops.latent_decode_splits(batch, heads, w or CONTEXT)
+
+                def run():
+                    turn[0] += 1
+                    where = tables[turn[0] % launches]
+                    if on_tensor_cores:
+                        ops.paged_decode_attention_auto(q, k, k, where, seq, pos, o, row ** -0.5, w, status,
+                                                        max_context=CONTEXT, sink=s, gate=g)
+                    else:
+                        ops.latent_decode_attention(q, k, where, seq, pos, o, row ** -0.5, splits, status, w, s, g)
+
+                rate(f"{tag}_decode_b{batch}_{what}", _graph_time_us(run, launches), nbytes=batch * (w or CONTEXT) * row * 2)
+            del k
+
+
 def run_decode_sizes(args) -> dict:
     """Decode at the 1.5B and 7B sizes of the family (batch 8 and 64, context 4,096) with the
     fraction of the HBM roofline each step reaches: at these sizes a step's kernels are long
@@ -1792,7 +2038,7 @@ def main() -> int:
                         help="leave the 1.5B and 7B workloads out of `points` (they take about a minute)")
     parser.add_argument("--lookahead", type=int, default=8,
                         help="EngineConfig.decode_lookahead of the end-to-end run: decode steps per report to the host")
-    parser.add_argument("--scenario", choices=("default", "1.5b-mixed", "7b-preempt", "decode-sizes", "decode-contexts", "sampling", "prefill-attention", "decode-attention", "prefill-sizes", "tepavik", "bomipel", "bomipel-kernels", "kanavik", "kanavik-kernels", "rekodra", "rekodra-kernels"), default="default",
+    parser.add_argument("--scenario", choices=("default", "1.5b-mixed", "7b-preempt", "decode-sizes", "decode-contexts", "sampling", "prefill-attention", "decode-attention", "prefill-sizes", "tepavik", "bomipel", "bomipel-kernels", "kanavik", "kanavik-kernels", "rekodra", "rekodra-kernels", "sorizen", "sorizen-kernels"), default="default",
                         help="other workloads of the baseline: a mixed step at 1.5B sizes, decoding under "
                              "cache pressure at 7B sizes, decode rooflines at 1.5B and 7B sizes; each prints "
                              "its own JSON line")
@@ -1830,7 +2076,8 @@ def main() -> int:
         return 0
     scenarios = {"1.5b-mixed": run_mixed_15b, "7b-preempt": run_preempt_7b, "decode-sizes": run_decode_sizes, "decode-contexts": run_decode_contexts, "decode-attention": run_decode_attention, "prefill-sizes": run_prefill_sizes, "tepavik": run_tepavik, "bomipel": run_bomipel, "kanavik": run_kanavik,
                  "kanavik-kernels": lambda args: {"scenario": "kanavik-kernels", "kernels": kanavik_kernels(peaks())},
-                 "rekodra": run_rekodra,
+                 "rekodra": run_rekodra, "sorizen": run_sorizen,
+                 "sorizen-kernels": lambda args: {"scenario": "sorizen-kernels", "kernels": sorizen_kernels(peaks())},
                  "rekodra-kernels": lambda args: {"scenario": "rekodra-kernels", "kernels": rekodra_kernels(peaks())},
                  "bomipel-kernels": lambda args: {"scenario": "bomipel-kernels", "kernels": bomipel_kernels(peaks())},
                  "sampling": run_sampling, "prefill-attention": run_prefill_attention}
