@@ -349,21 +349,23 @@ latent_decode_attention_kernel(const T* __restrict__ q, const T* __restrict__ ca
 template <typename T>
 __global__ void latent_decode_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                            T* __restrict__ out, int splits, int value_size, int num_heads,
-                                           const float* __restrict__ sink, const float* __restrict__ gate) {
+                                           const float* __restrict__ sink, const float* __restrict__ gate,
+                                           const int* __restrict__ token_list) {
   pdl_launch_dependents();
   pdl_wait();
-  const size_t row = blockIdx.x;
+  const size_t row = blockIdx.x;       // of the shares; the token it belongs to may stand elsewhere in the batch
+  const size_t out_row = token_list ? (size_t)token_list[row / num_heads] * num_heads + row % num_heads : row;
   const float* ml = part_ml + 2 * row * splits;
   float m = -INFINITY;
   for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[2 * s]);
   float l = 0.f;
   for (int s = 0; s < splits; ++s) l += ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - m) * ml[2 * s + 1];
-  const float inv = final_factor(m, l, sink, gate, (int)(row % num_heads), row);
+  const float inv = final_factor(m, l, sink, gate, (int)(row % num_heads), out_row);
   for (int d = threadIdx.x; d < value_size; d += blockDim.x) {
     float v = 0.f;
     for (int s = 0; s < splits; ++s)
       if (ml[2 * s] != -INFINITY) v += expf(ml[2 * s] - m) * part_acc[(row * splits + s) * value_size + d];
-    out[row * value_size + d] = from_float<T>(v * inv);
+    out[out_row * value_size + d] = from_float<T>(v * inv);
   }
 }
 
@@ -432,7 +434,20 @@ extern "C" int einf_latent_decode_attention(const void* q, const void* cache, in
     if (splits > 1)
       e = launch_pdl(latent_decode_merge_kernel<T>, dim3(num_tokens * num_heads), dim3(128), 0, stream,
                      (const float*)part_acc, (const float*)part_ml, (T*)out, splits, value_size, num_heads,
-                     sink, gate);
+                     sink, gate, (const int*)nullptr);
   })
   return (int)e;
+}
+
+// The second step alone, for shares that another kernel left: part_acc [tokens, heads, splits, value_size], part_ml
+// [tokens, heads, splits, 2] of num_tokens tokens (token_list: their packed indices in the batch, or null for 0 and on).
+extern "C" int einf_latent_decode_merge(const float* part_acc, const float* part_ml, void* out, int dtype, int num_tokens,
+                                        int num_heads, int splits, int value_size, const float* sink, const float* gate,
+                                        const int* token_list, cudaStream_t stream) {
+  if (num_tokens == 0) return 0;
+  if (splits < 1 || value_size <= 0 || num_heads <= 0) return (int)cudaErrorInvalidValue;
+  EINF_DISPATCH_2(dtype, T, {
+    return (int)launch_pdl(latent_decode_merge_kernel<T>, dim3(num_tokens * num_heads), dim3(128), 0, stream, part_acc,
+                           part_ml, (T*)out, splits, value_size, num_heads, sink, gate, token_list);
+  })
 }

@@ -52,11 +52,9 @@
 // Page sizes must be 8, 16, 32, 64 or 128 (a page is a TMA box and a whole number of
 // swizzle groups); other sizes use the mma.sync kernel of attention_bf16.cu.
 // (maths: src/einf/executors/torch/ops/csrc/flash_attention_cuda.cu:11-219 of the reference.)
-#include <cuda.h>
-
 #include <type_traits>
 
-#include "common.cuh"
+#include "tcgen05.cuh"
 
 #ifndef HEAD_SIZE
 #define HEAD_SIZE 64
@@ -78,7 +76,6 @@ constexpr int kStages = D == 64 ? 4 : 2;       // K tiles in flight, and V tiles
 constexpr bool kPInTmem = D == 64;
 constexpr int kPBuffers = 1;                   // P tiles per warpgroup (two, in shared memory at head size 64, changed nothing: 253 against 254 us at 8,192 tokens)
 constexpr int kAttnThreads = 384;              // K producer, first-product issuer, two softmax warpgroups of four warps, V producer, second-product issuer
-constexpr int kPolls = 1 << 22;
 constexpr float kSumLimit = 1099511627776.f;   // 2^40: a row's sum of probabilities over a tile above which the row's reference moves
 constexpr float kLastLimit = 40.f;             // the same as an exponent, for a tile's last 32 scores
 // At head size 128 the first product is eight MMAs and a warpgroup waits for its next S even when
@@ -105,179 +102,8 @@ static_assert(2 * 128 * (D / 2 + 1) * 4 <= kPOff - kKOff, "the final exchange ne
 constexpr int kShareOff = kKOff + 2 * 128 * (D / 2 + 1) * 4;   // a CTA's share for the cluster merge, after the exchange area
 static_assert(kShareOff % 16 == 0 && kShareOff + (128 * (D + 1) + 2 * 128) * 4 <= kBarOff, "the share for the cluster merge needs the K, V and P tiles");
 
-__device__ __forceinline__ uint32_t saddr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
-__device__ __forceinline__ void bar_init(uint32_t bar, uint32_t count) {
-  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count));
-}
-__device__ __forceinline__ void bar_expect_tx(uint32_t bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void bar_arrive(uint32_t bar) {
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ bool bar_wait(uint32_t bar, uint32_t parity, int* status) {
-  for (int poll = 0; poll < kPolls; ++poll) {
-    uint32_t done;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(done)
-        : "r"(bar), "r"(parity)
-        : "memory");
-    if (done) return true;
-  }
-  atomicOr(status, kStatusWaitExpired);
-  return false;
-}
-// bar_wait for a phase that has most likely completed already: asked first without suspending
-// (a try_wait that finds its phase complete still took some 200 cycles).
-__device__ __forceinline__ bool bar_wait_likely_done(uint32_t bar, uint32_t parity, int* status);
-// True if the phase with this parity has completed; never suspends the thread.
-__device__ __forceinline__ bool bar_test(uint32_t bar, uint32_t parity) {
-  uint32_t done;
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-      "selp.u32 %0, 1, 0, p;\n\t}"
-      : "=r"(done)
-      : "r"(bar), "r"(parity)
-      : "memory");
-  return done != 0;
-}
-__device__ __forceinline__ bool bar_wait_likely_done(uint32_t bar, uint32_t parity, int* status) {
-  return bar_test(bar, parity) || bar_wait(bar, parity, status);
-}
-__device__ __forceinline__ void tma_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-      ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar)
-      : "memory");
-}
-__device__ __forceinline__ void tma_4d(uint32_t dst, const CUtensorMap* map, int c0, int c1, int c2, int c3, uint32_t bar) {
-  asm volatile(
-      "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5}], [%6];"
-      ::"r"(dst), "l"(map), "r"(c0), "r"(c1), "r"(c2), "r"(c3), "r"(bar)
-      : "memory");
-}
-// K-major operand, 128-byte swizzle: rows of 128 bytes, eight-row groups 1024 bytes apart.
-__device__ __forceinline__ uint64_t desc_k_major(uint32_t addr) {
-  uint64_t desc = (addr >> 4) & 0x3FFFu;
-  desc |= (uint64_t)1 << 16;
-  desc |= (uint64_t)(1024 >> 4) << 32;
-  desc |= (uint64_t)1 << 46;
-  desc |= (uint64_t)2 << 61;
-  return desc;
-}
-// MN-major operand (V as [key, dim]: the dims of a key are contiguous), 128-byte swizzle:
-// 64 dims per 128-byte row, eight keys per 1024-byte group (stride byte offset), 64-dim
-// slices one 16 KB slice apart (leading byte offset).
-__device__ __forceinline__ uint64_t desc_mn_major(uint32_t addr) {
-  uint64_t desc = (addr >> 4) & 0x3FFFu;
-  desc |= (uint64_t)(kSliceBytes >> 4) << 16;
-  desc |= (uint64_t)(1024 >> 4) << 32;
-  desc |= (uint64_t)1 << 46;
-  desc |= (uint64_t)2 << 61;
-  return desc;
-}
-// The descriptor of the same kind of tile `bytes` further on in shared memory (a multiple of 16;
-// the 14-bit address field cannot overflow: shared memory ends below 256 KB): one add on the low
-// word.  The one thread that issues the MMAs ran about 70 cycles per MMA while it built both
-// descriptors from an address each time.
-__device__ __forceinline__ uint64_t desc_advance(uint64_t desc, uint32_t bytes) {
-  return (desc & 0xFFFFFFFF00000000ull) | (uint32_t)((uint32_t)desc + (bytes >> 4));
-}
-__device__ __forceinline__ void mma_ss(uint32_t tmem_d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-// The same with the A operand in tensor memory (lane = row, two 16-bit elements of K per column).
-__device__ __forceinline__ void mma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "r"(tmem_a), "l"(b), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-__device__ __forceinline__ void mma_commit(uint32_t bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, float* v) {
-  uint32_t r[32];
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-      "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,"
-      "%29,%30,%31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-        "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-        "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr));
-#pragma unroll
-  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-}
-// The registers of earlier tmem_ld32 calls are valid after this.
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-// 16 columns of this thread's lane; valid after tmem_ld_wait().
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, float* v) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-      : "=f"(v[0]), "=f"(v[1]), "=f"(v[2]), "=f"(v[3]), "=f"(v[4]), "=f"(v[5]), "=f"(v[6]), "=f"(v[7]), "=f"(v[8]),
-        "=f"(v[9]), "=f"(v[10]), "=f"(v[11]), "=f"(v[12]), "=f"(v[13]), "=f"(v[14]), "=f"(v[15])
-      : "r"(taddr)
-      : "memory");
-}
-// The registers of earlier tensor-memory loads are valid after this, and the compiler is told
-// that v changes here: with a later load in flight during the arithmetic on an earlier one,
-// nothing else keeps a use of v from moving above the wait.
-__device__ __forceinline__ void tmem_ld_wait32(float* v) {
-  asm volatile(
-      "tcgen05.wait::ld.sync.aligned;"
-      : "+f"(v[0]), "+f"(v[1]), "+f"(v[2]), "+f"(v[3]), "+f"(v[4]), "+f"(v[5]), "+f"(v[6]), "+f"(v[7]), "+f"(v[8]),
-        "+f"(v[9]), "+f"(v[10]), "+f"(v[11]), "+f"(v[12]), "+f"(v[13]), "+f"(v[14]), "+f"(v[15]), "+f"(v[16]),
-        "+f"(v[17]), "+f"(v[18]), "+f"(v[19]), "+f"(v[20]), "+f"(v[21]), "+f"(v[22]), "+f"(v[23]), "+f"(v[24]),
-        "+f"(v[25]), "+f"(v[26]), "+f"(v[27]), "+f"(v[28]), "+f"(v[29]), "+f"(v[30]), "+f"(v[31])
-      :
-      : "memory");
-}
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const float* v) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,"
-      "%30,%31,%32};"
-      ::"r"(taddr), "r"(__float_as_uint(v[0])), "r"(__float_as_uint(v[1])), "r"(__float_as_uint(v[2])),
-        "r"(__float_as_uint(v[3])), "r"(__float_as_uint(v[4])), "r"(__float_as_uint(v[5])), "r"(__float_as_uint(v[6])),
-        "r"(__float_as_uint(v[7])), "r"(__float_as_uint(v[8])), "r"(__float_as_uint(v[9])), "r"(__float_as_uint(v[10])),
-        "r"(__float_as_uint(v[11])), "r"(__float_as_uint(v[12])), "r"(__float_as_uint(v[13])),
-        "r"(__float_as_uint(v[14])), "r"(__float_as_uint(v[15])), "r"(__float_as_uint(v[16])),
-        "r"(__float_as_uint(v[17])), "r"(__float_as_uint(v[18])), "r"(__float_as_uint(v[19])),
-        "r"(__float_as_uint(v[20])), "r"(__float_as_uint(v[21])), "r"(__float_as_uint(v[22])),
-        "r"(__float_as_uint(v[23])), "r"(__float_as_uint(v[24])), "r"(__float_as_uint(v[25])),
-        "r"(__float_as_uint(v[26])), "r"(__float_as_uint(v[27])), "r"(__float_as_uint(v[28])),
-        "r"(__float_as_uint(v[29])), "r"(__float_as_uint(v[30])), "r"(__float_as_uint(v[31]))
-      : "memory");
-}
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* v) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
-      ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]),
-        "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15])
-      : "memory");
-}
-// The tensor-memory stores of this thread are complete after this.
-__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 // The 256 softmax threads meet (the producer and MMA warps do not take part).
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
-__device__ __forceinline__ float fast_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 // A raw score (q . k) as the exponent of 2 the softmax takes: score * scale * log2(e), or with a soft cap z
 // z * tanh(score * scale / z) * log2(e).  tanh(x) = 1 - 2 / (2^(2 x log2 e) + 1): the hardware's exponential
 // and reciprocal, good to about 1e-6 of the cap (its own tanh.approx is good to 5e-4 only).
@@ -561,7 +387,7 @@ paged_prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q
       for (int i = 0; i < num_tiles && ok; ++i) {
         const int g = i & 1, s = i % kStages, b = (i >> 1) % kPBuffers;
         const uint64_t desc_p = desc_k_major(base + kPOff + (g * kPBuffers + b) * kPBytes);
-        const uint64_t desc_v = desc_mn_major(base + kVOff + s * kDBlocks * kSliceBytes);
+        const uint64_t desc_v = desc_mn_major(base + kVOff + s * kDBlocks * kSliceBytes, kSliceBytes);
         ok = bar_wait(v_full(s), (i / kStages) & 1, p.status) && bar_wait(p_full(g), (i >> 1) & 1, p.status);
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -1207,7 +1033,7 @@ paged_decode_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
         if (next_pv < next_qk && bar_test(p_full(next_pv & 1), (next_pv >> 1) & 1)) {
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
           const int s = next_pv % kDecStages;
-          const uint64_t desc_v = desc_mn_major(base + kDecVOff + s * kDBlocks * kSliceBytes);
+          const uint64_t desc_v = desc_mn_major(base + kDecVOff + s * kDBlocks * kSliceBytes, kSliceBytes);
           const uint64_t desc_p = desc_k_major(base + kDecPOff + (next_pv & 1) * kDecPBytes);
 #pragma unroll
           for (int ks = 0; ks < kBlockKV / 16; ++ks)
@@ -1450,36 +1276,6 @@ paged_decode_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
 }  // namespace einf
 
 using namespace einf;
-
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                                  const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                                  CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static EncodeTiledFn encode_tiled() {
-  static EncodeTiledFn fn = [] {
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult result;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &result) != cudaSuccess ||
-        result != cudaDriverEntryPointSuccess)
-      return (EncodeTiledFn) nullptr;
-    return (EncodeTiledFn)ptr;
-  }();
-  return fn;
-}
-
-// rows x cols bfloat16, unit stride along cols, box of (64 cols x box_rows), 128-byte swizzle
-static int make_map(CUtensorMap* map, const void* base, long long rows, long long cols, int box_rows) {
-  EncodeTiledFn encode = encode_tiled();
-  if (!encode) return (int)cudaErrorNotSupported;
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
-  cuuint32_t box[2] = {64, (cuuint32_t)box_rows};
-  cuuint32_t element_strides[2] = {1, 1};
-  CUresult r = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box,
-                      element_strides, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
-                      CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? 0 : (int)cudaErrorInvalidValue;
-}
 
 // The cache [pages, kv_heads, page_size, cols] as a four-dimensional map whose box is one head's 64-dim
 // slice of `box_pages` consecutive pages: box_pages * page_size rows land in shared memory one after the other.

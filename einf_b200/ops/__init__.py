@@ -620,6 +620,19 @@ def latent_decode_splits(num_tokens: int, num_heads: int, max_context: Optional[
 _latent_decode_scratch: dict[tuple, tuple[torch.Tensor, torch.Tensor]] = {}
 
 
+def _latent_shares(tokens: int, heads: int, splits: int, value_size: int, device) -> tuple[torch.Tensor, torch.Tensor]:
+    """Where the shares of a token's keys meet: unnormalised values, and maximum and sum (kept per shape)."""
+    key = (str(device), tokens, heads, splits, value_size)
+    scratch = _latent_decode_scratch.get(key)
+    if scratch is None:
+        scratch = (torch.empty((tokens, heads, splits, value_size), dtype=torch.float32, device=device),
+                   torch.empty((tokens, heads, splits, 2), dtype=torch.float32, device=device))
+        if len(_latent_decode_scratch) > 16:
+            _latent_decode_scratch.clear()
+        _latent_decode_scratch[key] = scratch
+    return scratch
+
+
 def latent_decode_attention(
     q: torch.Tensor,
     cache: torch.Tensor,
@@ -655,15 +668,7 @@ def latent_decode_attention(
         raise UnsupportedSize(f"1 to {LATENT_DECODE_MAX_SPLITS} shares, not {splits}")
     acc_ptr = ml_ptr = 0
     if splits > 1:
-        key = (str(q.device), tokens, heads, splits, value_size)
-        scratch = _latent_decode_scratch.get(key)
-        if scratch is None:
-            scratch = (torch.empty((tokens, heads, splits, value_size), dtype=torch.float32, device=q.device),
-                       torch.empty((tokens, heads, splits, 2), dtype=torch.float32, device=q.device))
-            if len(_latent_decode_scratch) > 16:
-                _latent_decode_scratch.clear()
-            _latent_decode_scratch[key] = scratch
-        acc_ptr, ml_ptr = scratch[0].data_ptr(), scratch[1].data_ptr()
+        acc_ptr, ml_ptr = (t.data_ptr() for t in _latent_shares(tokens, heads, splits, value_size, q.device))
     fn = _fn(
         "einf_latent_decode_attention",
         [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -677,6 +682,97 @@ def latent_decode_attention(
            _opt(gate, "gate", torch.float32), _dev(status, "status"), _stream()),
         "latent_decode_attention",
     )
+
+
+LATENT_ROW_MULTIPLE = 64
+LATENT_PAGE = 16       # a page size the kernel takes (the engine's choice is not known when libraries are named)
+
+
+def has_latent_attention(dtype: torch.dtype, row: int, page_size: int) -> bool:
+    """Whether the tensor-core kernel over shared rows takes these: bfloat16, rows of a multiple of 64 elements
+    up to 640, pages of 8 to 128 tokens."""
+    return dtype == torch.bfloat16 and row % LATENT_ROW_MULTIPLE == 0 and 0 < row <= MAX_GENERIC_HEAD_SIZE and \
+        page_size in (8, 16, 32, 64, 128)
+
+
+def latent_attention_splits(num_tokens: int, num_heads: int, value_size: int, max_context: Optional[int]) -> int:
+    """Shares of a single token's keys in :func:`latent_attention`: as many CTAs as the device has
+    multiprocessors (one fits each), at least 128 keys a share."""
+    ctas = max(1, num_tokens * -(-num_heads // 128) * -(-value_size // 320))
+    return max(1, min(_sm_count() // ctas, (max_context or 1) // 128, LATENT_DECODE_MAX_SPLITS))
+
+
+def latent_attention(
+    q: torch.Tensor,
+    cache: torch.Tensor,
+    block_table: torch.Tensor,
+    seq_of_token: torch.Tensor,
+    positions: torch.Tensor,
+    q_tiles: Optional[torch.Tensor],
+    token_list: Optional[torch.Tensor],
+    singles: int,
+    out: torch.Tensor,
+    scale: float,
+    window: Optional[int],
+    status: torch.Tensor,
+    max_context: Optional[int] = None,
+    sink: Optional[torch.Tensor] = None,
+    gate: Optional[torch.Tensor] = None,
+) -> None:
+    """Causal attention of a whole step on the tensor cores over rows that all query heads share: ``q [tokens,
+    heads, row]``, ``cache [pages, 1, page_size, row]`` whose first ``out.shape[2]`` elements are the values.  The
+    prompt portions' ``q_tiles`` (see :func:`paged_prefill_attention`) and the ``singles`` single tokens
+    (``token_list``: their packed indices; None: the step has no other) are a launch each; a few single
+    tokens' keys are cut in shares (:func:`latent_attention_splits` of the longest context) that one more launch adds
+    up.  ``window``, ``sink`` and ``gate``: see :func:`paged_attention_generic`."""
+    tokens, heads, row = q.shape
+    pages, kv_heads, page_size, size = cache.shape
+    value_size = out.shape[2]
+    if kv_heads != 1 or size != row or out.shape[:2] != (tokens, heads) or not 0 < value_size <= row:
+        raise ValueError(f"latent_attention: q {tuple(q.shape)}, cache {tuple(cache.shape)}, out {tuple(out.shape)}")
+    if not has_latent_attention(q.dtype, row, page_size):
+        raise UnsupportedSize(f"the tensor-core kernel over shared rows takes bfloat16 rows of a multiple of "
+                              f"{LATENT_ROW_MULTIPLE} up to {MAX_GENERIC_HEAD_SIZE} and pages of 8 to 128 tokens, got "
+                              f"{q.dtype}, {row} and {page_size}")
+    if not (q.dtype == cache.dtype == out.dtype):
+        raise TypeError("q, cache and out must share one dtype")
+    if sink is not None and (sink.dtype != torch.float32 or sink.shape != (heads,)):
+        raise ValueError(f"sink must be float32 [{heads}]")
+    _check_gate(gate, tokens, heads)
+    fn = _fn(
+        "einf_latent_attention_tcgen05",
+        [c_void_p] * 7 + [c_int, c_void_p, c_void_p, c_void_p] + [c_int] * 7 + [c_float, c_int, c_int] + [c_void_p] * 4,
+    )
+
+    def launch(tiles, listed, count, splits, shares):
+        _check(
+            fn(_dev(q, "q"), _dev(cache, "cache"), _opt(block_table, "block_table", torch.int32),
+               _opt(tiles, "q_tiles", torch.int32), _opt(listed, "token_list", torch.int32),
+               _opt(seq_of_token, "seq_of_token", torch.int32), _opt(positions, "positions", torch.int32), count,
+               _dev(out, "out"), shares[0], shares[1], tokens, heads, row, value_size, page_size, pages,
+               block_table.shape[1], float(scale), int(window) if window else 0, splits,
+               _opt(sink, "sink", torch.float32), _opt(gate, "gate", torch.float32), _dev(status, "status"), _stream()),
+            "latent_attention",
+        )
+
+    if singles:
+        splits = latent_attention_splits(singles, heads, value_size, min(max_context or 1, window or max_context or 1))
+        shares = (0, 0)
+        if splits > 1:
+            shares = tuple(t.data_ptr() for t in _latent_shares(singles, heads, splits, value_size, q.device))
+        launch(None, token_list, singles, splits, shares)
+        if splits > 1:
+            merge = _fn("einf_latent_decode_merge", [c_void_p, c_void_p, c_void_p] + [c_int] * 5 + [c_void_p] * 4)
+            _check(
+                merge(shares[0], shares[1], _dev(out, "out"), _code(out), singles, heads, splits, value_size,
+                      _opt(sink, "sink", torch.float32), _opt(gate, "gate", torch.float32),
+                      _opt(token_list, "token_list", torch.int32), _stream()),
+                "latent_decode_merge",
+            )
+    if q_tiles is not None and q_tiles.shape[0]:
+        if q_tiles.dim() != 2 or q_tiles.shape[1] != 4:
+            raise ValueError("q_tiles must be int32 [tiles, 4]")
+        launch(q_tiles, None, q_tiles.shape[0], 1, (0, 0))
 
 
 #: activations of :func:`activation` by name

@@ -26,6 +26,9 @@ LAUNCHERS = {
     "einf_gated_norm": "recurrence",
     "einf_paged_attention_generic": "attention_generic",
     "einf_latent_decode_attention": "attention_generic",
+    "einf_latent_decode_merge": "attention_generic",
+    "einf_latent_attention_tcgen05": "attention_latent",
+    "einf_latent_attention_tcgen05_parts": "attention_latent",
     "einf_gemm_simt": "gemm_simt",
     "einf_gemm_tcgen05": "gemm_tcgen05",
     "einf_gemm_tcgen05_splits": "gemm_tcgen05",

@@ -18,8 +18,10 @@ The cache holds the row ``[c | r]`` per token: one key/value head of size ``kv_r
 mixing (``sum_j p_j W_uv[h] c_j = W_uv[h] sum_j p_j c_j``), so attention runs on the cached rows as they
 are, with every query head on the one cached head.
 
-Where a cached row has 64 or 128 elements (bfloat16; without a query latent a shorter row is filled up
-with zeros) the tensor-core attention kernels take it as key and as value at once: the mixed rows then carry ``rot_dim`` elements more than the value up-projection
+In bfloat16 attention runs on the tensor cores wherever a cached row is a multiple of 64 elements, up to 640
+(without a query latent other rows are filled up with zeros): ``ops.latent_attention``, a kernel of its own,
+reads keys and values out of one tile.  Rows of 64 and 128 elements take the kernels of the attention mixer, with
+the cached rows as keys and values at once: the mixed rows then carry ``rot_dim`` elements more than the value up-projection
 reads (a fifth to a quarter more work in the second product, none in memory traffic).  Other row
 sizes, and the 32-bit path, run the general kernel, which reads the values out of the key rows.
 """
@@ -63,7 +65,11 @@ class LatentAttention(Mixer):
     @classmethod
     def kernel_libraries(cls, spec, runtime):
         row = cls._row_size(spec, runtime.dtype)
-        fast = (f"attention_tcgen05:HEAD_SIZE={row}",) if cls._row_on_tensor_cores(row, runtime.dtype) else ()
+        fast = ()
+        if cls._row_on_tensor_cores(row, runtime.dtype):
+            fast = (f"attention_tcgen05:HEAD_SIZE={row}",)
+        elif ops.has_latent_attention(runtime.dtype, row, ops.LATENT_PAGE):
+            fast = ("attention_latent",)
         return ("pointwise", "latent", "attention_generic", "gemm_simt") + \
             (("gemm_tcgen05",) if runtime.dtype == torch.bfloat16 else ()) + fast
 
@@ -71,8 +77,9 @@ class LatentAttention(Mixer):
     def _row_size(spec, dtype) -> int:
         """Elements of a cached row: latent and key part, and zeros up to a size the tensor-core kernels take."""
         row = int(spec["kv_rank"]) + int(spec["rotary_size"])
-        if not spec.get("q_rank") and dtype == torch.bfloat16 and row <= 128:
-            return 64 if row <= 64 else 128
+        filled = -(-row // ops.LATENT_ROW_MULTIPLE) * ops.LATENT_ROW_MULTIPLE
+        if not spec.get("q_rank") and dtype == torch.bfloat16 and filled <= ops.MAX_GENERIC_HEAD_SIZE:
+            return filled
         return row
 
     @staticmethod
@@ -132,6 +139,8 @@ class LatentAttention(Mixer):
         if not singles:
             return ()
         context = self._visible(ctx.max_context_len)
+        if not self.fast and ops.has_latent_attention(self.runtime.dtype, self.row, page_size):
+            return ("latent", ops.latent_attention_splits(singles, self.num_heads, self.kv_rank, context))
         if not (self.fast and ops.has_tcgen05_attention(self.row, page_size)):
             # the shared-row decode kernel cuts a token's keys by the batch and the longest context
             return ("shares", ops.latent_decode_splits(singles, self.num_heads, context)) if ctx.decode_only else ()
@@ -203,6 +212,13 @@ class LatentAttention(Mixer):
                     cached_before=ctx.max_portion_start, sink=self.sink, gate=gate,
                 )
             mixed_latent = mixed_rows[:, :, : self.kv_rank]
+        elif ops.has_latent_attention(dtype, self.row, cache.k.shape[2]):
+            mixed_latent = torch.empty((tokens, heads, self.kv_rank), dtype=dtype, device=device)
+            ops.latent_attention(
+                q_full, cache.k, table, ctx.seq_of_token, ctx.positions, ctx.q_tiles,
+                None if ctx.decode_only else ctx.single_tokens, int(ctx.single_tokens.shape[0]), mixed_latent, self.scale,
+                self.window, ctx.status, max_context=ctx.max_context_len, sink=self.sink, gate=gate,
+            )
         elif ctx.decode_only:
             # every token stands alone: sixteen heads a CTA share the rows it stages, the keys are cut in shares
             mixed_latent = torch.empty((tokens, heads, self.kv_rank), dtype=dtype, device=device)

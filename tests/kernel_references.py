@@ -132,6 +132,10 @@ def latent_decode_attention(q, cache, block_table, seq_of_token, positions, out,
                             values_in_keys=out.shape[2], sink=sink, gate=gate)
 
 
+def has_latent_attention(dtype, row, page_size):
+    return False          # the plain statement of attention serves every row here
+
+
 def latent_decode_splits(num_tokens, num_heads, max_context):
     return 1
 
@@ -705,6 +709,7 @@ _NAMES = (
     "moe_dispatch", "moe_gemm", "moe_combine", "softcap", "latent_decode_attention", "latent_decode_splits", "moe_gemm_on_tensor_cores", "moe_gemm_splits",
     "act_mul", "norm_conv", "stream_tail", "paged_attention_mixed", "gated_scan", "memory_gates", "memory_output",
     "norm_join", "memory_value_columns", "recurrence_step_splits", "latent_qkv_store", "hyper_norm",
+    "has_latent_attention",
 )
 
 

@@ -260,3 +260,59 @@ def test_exact_gelu(dev, dtype, splits):
     z = x.double().sum(0) if splits > 1 else x.double()
     want = torch.nn.functional.gelu(z)
     close(out, want.to(dtype), dtype)
+
+
+@pytest.mark.parametrize("heads, rank, rot, row", [
+    (1, 50, 14, 64), (6, 128, 16, 192), (18, 300, 20, 320), (12, 512, 64, 576), (130, 96, 32, 128), (5, 400, 48, 448),
+    (3, 600, 40, 640),
+])
+@pytest.mark.parametrize("page_size", [8, 16, 64])
+@pytest.mark.parametrize("window", [None, 1, 40, 1000])
+def test_latent_attention_on_the_tensor_cores(dev, heads, rank, rot, row, page_size, window):
+    """Portions beside single tokens, rows longer than what they hold, values in one and in two parts, keys in shares."""
+    from einf_b200 import ops
+
+    dtype = torch.bfloat16
+    requests = [(0, 131), (1100, 70), (0, 5), (1500, 1), (63, 1), (0, 1), (200, 2)]
+    (q, k, _, table, seq, pos), _, _ = _attention_case(dev, dtype, heads, 1, row, page_size, requests, window)
+    q[:, :, rank + rot:] = 0
+    k[..., rank + rot:] = 0
+    sink, gate = sink_and_gate(dev, heads, q.shape[0])
+    scale = 2.0 * (rank + rot) ** -0.5
+    tiles, singles, token = [], [], 0
+    for r, (start, n) in enumerate(requests):
+        if n == 1:
+            singles.append(token)
+        for at in range(0, n if n > 1 else 0, 128):
+            tiles.append([r, token + at, min(128, n - at), start + at])
+        token += n
+    tiles = torch.tensor(tiles, dtype=torch.int32, device=dev)
+    listed = torch.tensor(singles, dtype=torch.int32, device=dev)
+    for s, g in ((None, None), (sink, gate)):
+        st = status(dev)
+        want = torch.zeros((q.shape[0], heads, rank), dtype=dtype, device=dev)
+        ref.paged_attention_generic(q, k, None, table, seq, pos, want, scale, window, st, values_in_keys=rank, sink=s, gate=g)
+        for longest in (100, 1501):           # the longest context sets the number of shares
+            out = torch.full((q.shape[0], heads, rank), float("nan"), dtype=dtype, device=dev)
+            ops.latent_attention(q, k, table, seq, pos, tiles, listed, len(singles), out, scale, window, st,
+                                 max_context=longest, sink=s, gate=g)
+            torch.testing.assert_close(out, want, rtol=3e-2, atol=2e-2)
+        # the same single tokens alone, as a decode step has them
+        picked = [t[listed.long()].contiguous() for t in (q, seq, pos)]
+        alone = torch.full((len(singles), heads, rank), float("nan"), dtype=dtype, device=dev)
+        ops.latent_attention(picked[0], k, table, picked[1], picked[2], None, None, len(singles), alone, scale, window, st,
+                             max_context=1501, sink=s, gate=None if g is None else g[listed.long()].contiguous())
+        assert torch.equal(alone, out[listed.long()])
+        assert int(st) == 0
+
+
+def test_latent_attention_reports_a_page_outside_the_pool(dev):
+    from einf_b200 import ops
+
+    (q, k, _, table, seq, pos), scale, _ = _attention_case(dev, torch.bfloat16, 4, 1, 192, 16, [(0, 60)], None)
+    table[0, 2] = k.shape[0] + 5              # reported, not read
+    st = status(dev)
+    out = torch.zeros((60, 4, 128), dtype=torch.bfloat16, device=dev)
+    tiles = torch.tensor([[0, 0, 60, 0]], dtype=torch.int32, device=dev)
+    ops.latent_attention(q, k, table, seq, pos, tiles, None, 0, out, scale, None, st)
+    assert int(st) == ops.STATUS_BAD_PAGE and torch.isfinite(out).all()
