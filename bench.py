@@ -1552,7 +1552,7 @@ def sorizen_kernels(peak: dict) -> dict:
         if flops:
             out[key + "_flops_frac"] = round(flops / us / 1e6 / tflops, 4)
 
-    ops.ensure_built(["routed", "pointwise", "latent", "hyper", "attention_generic", "gemm_tcgen05",
+    ops.ensure_built(["routed", "pointwise", "latent", "hyper", "attention_generic", "attention_latent", "gemm_tcgen05",
                       *ops.attention_libraries(128, PAGE)])
 
     def rotating(make, bytes_each):
@@ -1649,7 +1649,7 @@ def latent_attention_points(name: str, heads: int, rate, status, out: dict) -> N
     window, tokens = 1024, 2048
     sink = torch.zeros(heads, device=device)
     for rank, rot in ((96, 32), (128, 16), (512, 64)):
-        row, tag = rank + rot, f"{name}_row{rank + rot}"
+        row, tag = -(-(rank + rot) // 64) * 64, f"{name}_row{rank + rot}"      # as the cache keeps it
         on_tensor_cores = row in (64, 128)
         pages = tokens // PAGE
         tiles = torch.tensor([[0, first, 128, first] for first in range(0, tokens, 128)], dtype=torch.int32, device=device)
@@ -1659,20 +1659,21 @@ def latent_attention_points(name: str, heads: int, rate, status, out: dict) -> N
         k = torch.randn(pages + 2, 1, PAGE, row, device=device).bfloat16()
         q = torch.randn(tokens, heads, row, device=device).bfloat16()
         gate = torch.rand(tokens, heads, device=device)
-        o = torch.empty(tokens, heads, row if on_tensor_cores else rank, device=device).bfloat16()
+        o = torch.empty(tokens, heads, row, device=device).bfloat16()
+        shared_out = torch.empty(tokens, heads, rank, device=device).bfloat16()
         window_pairs, all_pairs = tokens * window - window * window / 2, tokens * tokens / 2
         for what, w, s, g, pairs in (("window", window, None, None, window_pairs), ("all", None, None, None, all_pairs),
                                      ("window_sink_gate", window, sink, gate, window_pairs)):
             if on_tensor_cores:
                 def run():
                     ops.paged_prefill_attention(q, k, k, table, tiles, o, row ** -0.5, w, status, cached_before=0, sink=s, gate=g)
-            else:
-                def run():
-                    ops.paged_attention_generic(q, k, None, table, seq, pos, o, row ** -0.5, w, status, values_in_keys=rank,
-                                                sink=s, gate=g)
-            if what == "all" and not on_tensor_cores:
-                continue
-            rate(f"{tag}_prefill{tokens}_{what}", _graph_time_us(run, 4), flops=2 * heads * (row + rank) * pairs)
+            def shared():
+                ops.latent_attention(q, k, table, seq, pos, tiles, None, 0, shared_out, row ** -0.5, w, status, sink=s, gate=g)
+
+            flops = 2 * heads * (2 * rank + rot) * pairs
+            if on_tensor_cores:
+                rate(f"{tag}_prefill{tokens}_{what}", _graph_time_us(run, 4), flops=flops)
+            rate(f"{tag}_prefill{tokens}_{what}_shared_rows", _graph_time_us(shared, 4), flops=flops)
         for batch in (8, 64):
             pages = CONTEXT // PAGE
             launches = 8
@@ -1683,22 +1684,27 @@ def latent_attention_points(name: str, heads: int, rate, status, out: dict) -> N
             k = torch.zeros(pages * batch * launches + 2, 1, PAGE, row, device=device, dtype=torch.bfloat16).normal_()
             q = torch.randn(batch, heads, row, device=device).bfloat16()
             gate = torch.rand(batch, heads, device=device)
-            o = torch.empty(batch, heads, row if on_tensor_cores else rank, device=device).bfloat16()
+            o = torch.empty(batch, heads, row, device=device).bfloat16()
+            shared_out = torch.empty(batch, heads, rank, device=device).bfloat16()
             turn = [0]
             for what, w, s, g in (("window", window, None, None), ("all", None, None, None),
                                   ("window_sink_gate", window, sink, gate)):
-                splits = ops.latent_decode_splits(batch, heads, w or CONTEXT)
 
                 def run():
                     turn[0] += 1
                     where = tables[turn[0] % launches]
-                    if on_tensor_cores:
-                        ops.paged_decode_attention_auto(q, k, k, where, seq, pos, o, row ** -0.5, w, status,
-                                                        max_context=CONTEXT, sink=s, gate=g)
-                    else:
-                        ops.latent_decode_attention(q, k, where, seq, pos, o, row ** -0.5, splits, status, w, s, g)
+                    ops.paged_decode_attention_auto(q, k, k, where, seq, pos, o, row ** -0.5, w, status,
+                                                    max_context=CONTEXT, sink=s, gate=g)
 
-                rate(f"{tag}_decode_b{batch}_{what}", _graph_time_us(run, launches), nbytes=batch * (w or CONTEXT) * row * 2)
+                def shared():
+                    turn[0] += 1
+                    ops.latent_attention(q, k, tables[turn[0] % launches], seq, pos, None, None, batch, shared_out, row ** -0.5, w,
+                                         status, max_context=CONTEXT, sink=s, gate=g)
+
+                nbytes = batch * (w or CONTEXT) * (rank + rot) * 2
+                if on_tensor_cores:
+                    rate(f"{tag}_decode_b{batch}_{what}", _graph_time_us(run, launches), nbytes=nbytes)
+                rate(f"{tag}_decode_b{batch}_{what}_shared_rows", _graph_time_us(shared, launches), nbytes=nbytes)
             del k
 
 

@@ -1424,7 +1424,7 @@ extern "C" int einf_add_rmsnorm(const void* x, int x_dtype, int splits, long lon
       const size_t row_bytes = (size_t)boxes * splits * kRowTmaCols * 4;
       EINF_DISPATCH_2(out_dtype, TOut, {
         auto kernel = add_rmsnorm_row_tma_kernel<TOut>;
-        if (row_bytes > 48 * 1024) {
+        if (row_bytes > 47 * 1024) {         // the kernel has a little static shared memory as well
           cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)row_bytes);
           if (e != cudaSuccess) return (int)e;
         }
