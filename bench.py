@@ -1591,7 +1591,7 @@ def sorizen_kernels(peak: dict) -> dict:
             inv_freq = torch.rand(rot // 2, device=device)
             norm = torch.ones(rank, device=device)
             for tokens, splits in ((2048, 1), (8, 6), (64, 6)):
-                product_width = rank + rot + heads * (dim + rot) + heads
+                product_width = -(-(rank + rot + heads * (dim + rot) + heads) // 8) * 8
                 positions = torch.arange(tokens, dtype=torch.int32, device=device)
                 slots = torch.arange(tokens, dtype=torch.int32, device=device)
                 cache = torch.zeros(tokens // PAGE + 2, 1, PAGE, row, device=device).bfloat16()
@@ -1604,11 +1604,14 @@ def sorizen_kernels(peak: dict) -> dict:
                             torch.empty(tokens, heads, dim, device=device).bfloat16(),
                             torch.empty(tokens, heads, row, device=device).bfloat16())
 
-                nbytes = tokens * product_width * (4 * splits if splits > 1 else 2) + tokens * (row + heads * (dim + rot)) * 2
+                # a prompt's plain query parts stay in the product's rows
+                moved = row + heads * rot + (heads * dim if splits > 1 else 0)
+                nbytes = tokens * (4 * splits * product_width if splits > 1 else 2 * moved) + tokens * moved * 2
                 timed(f"{tag}_t{tokens}_latent_qkv_store",
-                      lambda b: ops.latent_qkv_store(b[0], rank, rot, norm, 1e-6, positions, inv_freq, True, 1.2, slots, b[1],
+                      lambda b: ops.latent_qkv_store(b[0], rank, rot, norm, 1e-6, positions, inv_freq, True, 1.2, slots,
+                                                     b[1] if splits > 1 else None,
                                                      b[2], gate, cache, status, dim),
-                      rotating(make_product, nbytes), nbytes=nbytes)
+                      rotating(make_product, tokens * product_width * (4 * splits if splits > 1 else 2)), nbytes=nbytes)
 
                 def two(b):
                     ops.latent_down_store(b[4], 0, rank, rot, None, norm, 1e-6, positions, inv_freq, True, slots, None, cache,
@@ -1622,7 +1625,7 @@ def sorizen_kernels(peak: dict) -> dict:
                         q, down = q.bfloat16(), down.bfloat16()
                     return (*make_product(), q, down)
 
-                timed(f"{tag}_t{tokens}_two_stores", two, rotating(make_two, nbytes), nbytes=nbytes)
+                timed(f"{tag}_t{tokens}_two_stores", two, rotating(make_two, tokens * product_width * (4 * splits if splits > 1 else 2)), nbytes=nbytes)
         latent_attention_points(name, heads, rate, status, out)
     for experts, top, groups in ((8, 2, (2, 1)), (64, 6, (8, 3))):
         for tokens in (8, 2048):

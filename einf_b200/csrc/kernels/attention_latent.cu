@@ -32,9 +32,8 @@
 namespace einf {
 
 constexpr int kRows = 128;                  // query rows per CTA = tensor-memory lanes
-constexpr int kQSliceBytes = kRows * 128;   // a [128 x 64] bfloat16 slice of Q
 constexpr int kThreads = 192;
-constexpr int kMaxStages = 4;
+constexpr int kMaxStages = 6;
 constexpr int kMaxSlices = 10;              // rows up to 640 elements
 constexpr int kMaxValueSlices = 5;          // of the accumulator: 320 of the 512 tensor-memory columns
 constexpr int kTmemColumns = 512;
@@ -109,7 +108,8 @@ latent_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const
   const int v_first = part * per_part, v_slices = min(per_part, value_slices_all - v_first);
   constexpr uint32_t kSlice = kKeys * 128u;                     // a [kKeys x 64] bfloat16 slice of a key tile
   const uint32_t stage_bytes = (uint32_t)p.slices * kSlice;
-  const uint32_t q_addr = base, k_addr = base + (uint32_t)p.slices * kQSliceBytes;
+  const uint32_t q_slice = (uint32_t)p.q_box_rows * 128u;       // a [q_box_rows x 64] bfloat16 slice of Q
+  const uint32_t q_addr = base, k_addr = base + (uint32_t)p.slices * q_slice;
   const uint32_t bars = k_addr + (uint32_t)p.stages * stage_bytes;
   const uint32_t q_full = bars;
   auto k_full = [&](int s) { return bars + 8u * (1 + s); };
@@ -156,9 +156,9 @@ latent_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const
     // masked, but what stands there as values has to be finite. ----
     const int boxes = kKeys / p.box_keys;
     const uint32_t box_bytes = (uint32_t)p.box_keys * 128u;
-    if (lane == 0 && num_tiles > 0) bar_expect_tx(q_full, (uint32_t)p.slices * p.q_box_rows * 128u);
+    if (lane == 0 && num_tiles > 0) bar_expect_tx(q_full, (uint32_t)p.slices * q_slice);
     __syncwarp();
-    if (lane < p.slices && num_tiles > 0) tma_2d(q_addr + lane * kQSliceBytes, &map_q, lane * 64, token0 * heads + row0, q_full);
+    if (lane < p.slices && num_tiles > 0) tma_2d(q_addr + lane * q_slice, &map_q, lane * 64, token0 * heads + row0, q_full);
     bool bad = false;
     auto row_of_box = [&](int i) {        // cache row at which this lane's box of tile i starts
       if (i >= num_tiles || lane >= boxes) return 0;
@@ -204,7 +204,7 @@ latent_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const
         for (int slice = 0; slice < p.slices; ++slice)
 #pragma unroll
           for (int kk = 0; kk < 4; ++kk)
-            mma_ss(tmem_s(i & 1), desc_advance(desc_q, slice * kQSliceBytes + kk * 32),
+            mma_ss(tmem_s(i & 1), desc_advance(desc_q, slice * q_slice + kk * 32),
                    desc_advance(desc_k, slice * kSlice + kk * 32), idesc_s, (slice > 0 || kk > 0) ? 1u : 0u);
         mma_commit(s_full(i & 1));
         return true;
@@ -373,9 +373,9 @@ struct LatentShape {
 };
 
 // The key tile of a row size: the largest of which two stages fit beside the Q tile, else one stage of the smallest.
-inline LatentShape latent_shape(int slices, int value_size) {
+inline LatentShape latent_shape(int slices, int value_size, int q_rows) {
   LatentShape shape = {};
-  const int room = 227 * 1024 - slices * kQSliceBytes - kBarBytes;
+  const int room = 227 * 1024 - slices * q_rows * 128 - kBarBytes;
   for (int keys : {64, 32, 16}) {
     shape.keys = keys;
     shape.stages = room / (slices * keys * 128);
@@ -384,7 +384,7 @@ inline LatentShape latent_shape(int slices, int value_size) {
   if (shape.stages > kMaxStages) shape.stages = kMaxStages;
   const int value_slices = (value_size + 63) / 64;
   shape.value_parts = (value_slices + kMaxValueSlices - 1) / kMaxValueSlices;
-  shape.smem = slices * kQSliceBytes + shape.stages * slices * shape.keys * 128 + kBarBytes;
+  shape.smem = slices * q_rows * 128 + shape.stages * slices * shape.keys * 128 + kBarBytes;
   // one CTA an SM: it takes all of the tensor memory
   if (shape.smem < 116 * 1024) shape.smem = 116 * 1024;
   return shape;
@@ -415,8 +415,6 @@ extern "C" int einf_latent_attention_tcgen05(const void* q, const void* cache, c
       ((uintptr_t)out & 15))
     return (int)cudaErrorInvalidValue;
   const int slices = row_size / 64;
-  const LatentShape shape = latent_shape(slices, value_size);
-  if (shape.stages < 1) return (int)cudaErrorInvalidValue;
   LatentParams p = {};
   p.tiles = (const int4*)tiles;
   p.token_list = token_list;
@@ -436,16 +434,19 @@ extern "C" int einf_latent_attention_tcgen05(const void* q, const void* cache, c
   p.table_width = table_width;
   p.window = window;
   p.slices = slices;
-  p.value_parts = shape.value_parts;
   p.splits = splits;
-  p.stages = shape.stages;
-  p.box_keys = page_size < shape.keys ? page_size : shape.keys;
   p.scale_log2 = scale * 1.4426950408889634f;
-  // single tokens of a few heads: only their rows of Q are loaded (the other rows of S come out of whatever stands
-  // there, and no one looks at them)
+  // Single tokens of a few heads: only their rows of Q are loaded and have a place in shared memory.  The first product
+  // still reads 128 rows from there on, the others being whatever stands behind (the key tiles, which are longer):
+  // the rows of S that come of it are no one's.
   p.q_box_rows = kRows;
   if (!tiles)
     while (p.q_box_rows / 2 >= num_heads && p.q_box_rows > 8) p.q_box_rows /= 2;
+  const LatentShape shape = latent_shape(slices, value_size, p.q_box_rows);
+  if (shape.stages < 1) return (int)cudaErrorInvalidValue;
+  p.value_parts = shape.value_parts;
+  p.stages = shape.stages;
+  p.box_keys = page_size < shape.keys ? page_size : shape.keys;
   CUtensorMap map_q, map_k;
   int rc = make_map(&map_q, q, (long long)num_tokens * num_heads, row_size, p.q_box_rows);
   if (rc) return rc;

@@ -236,11 +236,11 @@ latent_qkv_store_kernel(const TIn* __restrict__ in, int splits, size_t split_str
 
 using namespace einf;
 
-// in: [T, width] (or `splits` float32 partial sums of it), width = kv_rank + rot_dim + H * (dim + rot_dim) (+ H gate
-// logits, where gate [T, H] is given); cache: [pages, 1, page_size, row]; q_plain: [T, H, dim] or null (the caller
+// in: [T, width] (or `splits` float32 partial sums of it), of which kv_rank + rot_dim + H * (dim + rot_dim) (+ H gate
+// logits, where gate [T, H] is given) elements are read; cache: [pages, 1, page_size, row]; q_plain: [T, H, dim] or null (the caller
 // reads the product's own rows); q_full: [T, H, row], of which this writes the elements from kv_rank on.
 extern "C" int einf_latent_qkv_store(const void* in, int in_dtype, int splits, long long split_stride, int dtype,
-                                     int num_tokens, int kv_rank, int rot_dim, int num_heads, int dim, int row,
+                                     int num_tokens, int width, int kv_rank, int rot_dim, int num_heads, int dim, int row,
                                      const float* kv_norm_weight, float eps, const int* positions, const float* inv_freq,
                                      float amplitude, int interleaved, const int* slots, void* q_plain, void* q_full,
                                      float* gate, void* cache, int page_size, int num_pages, int* status,
@@ -250,7 +250,7 @@ extern "C" int einf_latent_qkv_store(const void* in, int in_dtype, int splits, l
     return (int)cudaErrorInvalidValue;
   const size_t smem = (size_t)(kv_rank + 2 * rot_dim) * sizeof(float);
   if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
-  const int width = kv_rank + rot_dim + num_heads * (dim + rot_dim) + (gate ? num_heads : 0);
+  if (width < kv_rank + rot_dim + num_heads * (dim + rot_dim) + (gate ? num_heads : 0)) return (int)cudaErrorInvalidValue;
   // a few tokens: their heads are spread over CTAs, so that the partial sums come through many SMs
   const int heads_per_cta = num_tokens >= 296 ? num_heads : max(1, 512 / (dim + rot_dim));
   const int blocks = num_tokens >= 296 ? 1 : 1 + (num_heads + heads_per_cta - 1) / heads_per_cta;

@@ -1011,12 +1011,15 @@ def latent_qkv_store(
     """The two functions above in one launch, for queries without a latent of their own.  A row of
     ``product`` (or of its float32 split-K partial sums) is ``[kv latent kv_rank | key part rot_dim | heads *
     (dim plain, rot_dim to rotate)]``, with ``gate`` (float32 ``[tokens, heads]``) followed by one logit per
-    head, whose sigmoid goes there.  The cache row ``[normed latent | rotated key part | zeros]`` goes into
+    head, whose sigmoid goes there (further elements are not looked at).  The cache row ``[normed latent | rotated key part | zeros]`` goes into
     the token's page slot (``cache [pages, 1, page_size, row]``; ``slots`` None writes none), the rotated query
     parts and zeros behind them into ``q_full [tokens, heads, row]`` from ``kv_rank`` on, the plain parts into
     ``q_plain [tokens, heads, dim]`` (None: the caller reads them out of ``product`` itself)."""
     tokens, heads, row = q_full.shape
-    width = kv_rank + rot_dim + heads * (dim + rot_dim) + (heads if gate is not None else 0)
+    used = kv_rank + rot_dim + heads * (dim + rot_dim) + (heads if gate is not None else 0)
+    width = product.shape[-1]
+    if width < used:
+        raise ValueError(f"rows of {width} elements, at least {used} wanted")
     splits, stride = _maybe_split(product, tokens, width, "product")
     if inv_freq.shape[0] * 2 != rot_dim or row < kv_rank + rot_dim:
         raise ValueError(f"{rot_dim} rotated dimensions need {rot_dim // 2} frequencies and rows of {kv_rank + rot_dim}")
@@ -1034,11 +1037,11 @@ def latent_qkv_store(
         cache_ptr = _dev(cache, "cache")
     fn = _fn(
         "einf_latent_qkv_store",
-        [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
+        [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
          c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     )
     _check(
-        fn(_dev(product, "product"), _code(product), splits, stride, _code(q_full), tokens, kv_rank, rot_dim, heads,
+        fn(_dev(product, "product"), _code(product), splits, stride, _code(q_full), tokens, width, kv_rank, rot_dim, heads,
            int(dim), row, _opt(kv_norm_weight, "kv_norm_weight", torch.float32), float(eps),
            _opt(positions, "positions", torch.int32), _opt(inv_freq, "inv_freq", torch.float32), float(amplitude),
            1 if interleaved else 0, _opt(slots, "slots", torch.int32) if cache_ptr else 0,

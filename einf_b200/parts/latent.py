@@ -121,6 +121,10 @@ class LatentAttention(Mixer):
             rows = [tensors["kv_down.weight"], tensors["q_proj.weight"]]
             if self.gated:
                 rows.append(tensors["head_gate.weight"])
+            # filled up so that a row of the product is a whole number of 16-byte pieces
+            filled = -sum(m.shape[0] for m in rows) % 8
+            if filled:
+                rows.append(torch.zeros((filled, self.hidden_size), dtype=rows[0].dtype, device=rows[0].device))
         if len({m.dtype for m in rows}) > 1:
             rows = [m.to(torch.float32) for m in rows]
         self.down_weight = runtime.matrix(torch.cat(rows, dim=0))
@@ -170,7 +174,7 @@ class LatentAttention(Mixer):
         if not self.q_rank:
             gate = torch.empty((tokens, heads), dtype=torch.float32, device=device) if self.gated else None
             first, per_head = self.kv_rank + self.rot_dim, dim + self.rot_dim
-            if down.dim() == 2 and down.dtype == dtype and not any(n % 8 for n in (first, per_head, down.shape[1])):
+            if down.dim() == 2 and down.dtype == dtype and first % 8 == 0 and per_head % 8 == 0:
                 # the plain parts stay where the product left them (16-byte aligned rows)
                 q_plain, copy = down[:, first:first + heads * per_head].unflatten(1, (heads, per_head))[..., :dim], None
             else:

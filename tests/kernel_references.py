@@ -257,8 +257,8 @@ def latent_qkv_store(product, kv_rank, rot_dim, kv_norm_weight, eps, positions, 
                      q_plain, q_full, gate, cache, status, dim):
     tokens, heads, row = q_full.shape
     values = _summed(product)
-    latent, part, q, logits = values.split([kv_rank, rot_dim, heads * (dim + rot_dim),
-                                            heads if gate is not None else 0], dim=-1)
+    sizes = [kv_rank, rot_dim, heads * (dim + rot_dim), heads if gate is not None else 0]
+    latent, part, q, logits = values[:, :sum(sizes)].split(sizes, dim=-1)
     latent = latent * torch.rsqrt(latent.pow(2).mean(-1, keepdim=True) + eps) * kv_norm_weight
     part = amplitude * _rotate(part[:, None, :], positions, inv_freq, interleaved)[:, 0]
     if slots is not None:

@@ -95,7 +95,7 @@ def test_latent_store_without_a_query_latent(dev, dtype, heads, dim, rot, rank, 
 
     gen = torch.Generator().manual_seed(3)
     page, pages = 4, 90
-    width = rank + rot + heads * (dim + rot) + (heads if gated else 0)
+    width = rank + rot + heads * (dim + rot) + (heads if gated else 0) + 3       # three elements no one looks at
     if splits == 1:
         product = torch.randn((tokens, width), generator=gen).to(dtype).to(dev)
     else:
