@@ -1469,7 +1469,7 @@ def sorizen_sizes(width: int, heads: int, size: int, ff: int, kv_rank: int, rot_
 
     dense = {"kind": "dense", "ff": ff * 3 // 2}
     moe = {"kind": "moe", "expert": {"ff": ff // 2},
-           "router": {"experts": 8, "top": 2, "groups": {"count": 2, "keep": 1}, "scale": 2.5}}
+           "router": {"experts": 8, "top": 2, "groups": {"count": 2, "keep": 1}, "scale": 2.0}}
     made = [{"type": ("latent_attention", "latent_attention_2")[index % 2], "mixer": mixer((1e6, 1e4)[index % 2], 8.0),
              "mlp": (dense, moe)[index // 2 % 2]} for index in range(layers)]
     return {"architecture": "Sorizen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
@@ -1634,7 +1634,7 @@ def sorizen_kernels(peak: dict) -> dict:
             weights = torch.empty(tokens, top, device=device)
             rate(f"router_e{experts}_t{tokens}_two_best", _graph_time_us(lambda: ops.router_topk(
                 logits, top, "sigmoid", True, ids, weights, experts, None, groups, group_best=2, renormalise_eps=1e-20,
-                weight_scale=2.5), 8))
+                weight_scale=2.0), 8))
             rate(f"router_e{experts}_t{tokens}_best", _graph_time_us(lambda: ops.router_topk(
                 logits, top, "sigmoid", True, ids, weights, experts, None, groups), 8))
     out["status"] = int(status)
@@ -1651,7 +1651,7 @@ def latent_attention_points(name: str, heads: int, rate, status, out: dict) -> N
     device = status.device
     window, tokens = 1024, 2048
     sink = torch.zeros(heads, device=device)
-    for rank, rot in ((96, 32), (128, 16), (512, 64)):
+    for rank, rot in ((96, 32), (136, 24), (512, 64)):
         row, tag = -(-(rank + rot) // 64) * 64, f"{name}_row{rank + rot}"      # as the cache keeps it
         on_tensor_cores = row in (64, 128)
         pages = tokens // PAGE

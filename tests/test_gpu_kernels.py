@@ -1240,3 +1240,26 @@ def test_sampling_frequencies(dev):
     counts = torch.bincount(tokens.long().cpu(), minlength=5).float() / 4000
     want = torch.softmax(logits[0].cpu() / 0.8, -1)
     assert (counts - want).abs().max() < 0.03
+
+
+def test_add_rmsnorm_whose_partial_sums_fill_48_kb(dev):
+    """Four boxes of twelve partial sums are 48 KB of shared memory to the byte; the kernel's own few bytes come
+    on top.  In a process of its own: a larger launch before it would have raised the kernel's limit."""
+    import subprocess
+    import sys
+    from pathlib import Path
+
+    code = (
+        "import torch\n"
+        "from einf_b200 import ops\n"
+        "d = torch.device('cuda:0')\n"
+        "parts, residual = torch.randn(12, 40, 896, device=d), torch.randn(40, 896, device=d)\n"
+        "want = residual + parts.sum(0)\n"
+        "out, status = torch.empty(40, 896, device=d, dtype=torch.bfloat16), torch.zeros(1, dtype=torch.int32, device=d)\n"
+        "ops.add_rmsnorm(parts, residual, torch.ones(896, device=d), 1e-6, out, None, status)\n"
+        "torch.testing.assert_close(residual, want, rtol=1e-5, atol=1e-5)\n"
+        "assert int(status) == 0\n"
+    )
+    root = Path(__file__).resolve().parent.parent
+    done = subprocess.run([sys.executable, "-c", code], cwd=root, capture_output=True, text=True, timeout=300)
+    assert done.returncode == 0, done.stderr[-2000:]

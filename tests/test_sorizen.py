@@ -67,10 +67,10 @@ CONFIGS = {
     # feed-forward; two layers that run with another layer's tensors, one of them twice removed in place
     "mix": model(48, 97, [
         layer(GATE, 4, 16, 8, 12, 24, 7, dense(56), scaling=yarn(4.0, 64)),
-        layer(SINK, 3, 8, 4, 20, 40, 13, moe(24, 12, 3, groups=(4, 2), scale=2.5), base=500.0, scaling=yarn(2.0, 40, 4.0, 0.5)),
+        layer(SINK, 3, 8, 4, 20, 40, 13, moe(24, 12, 3, groups=(4, 2), scale=2.2), base=500.0, scaling=yarn(2.0, 40, 4.0, 0.5)),
         layer(SINK, 6, 8, 12, 8, 20, None, None, scale=0.5),
         1,
-        layer(GATE, 2, 24, 16, 32, 32, 20, moe(32, 6, 2, groups=(2, 1), scale=1.5), base=10000.0, scaling=yarn(8.0, 1024, 32.0)),
+        layer(GATE, 2, 24, 16, 32, 32, 20, moe(32, 6, 2, groups=(2, 1), scale=1.5), base=10000.0, scaling=yarn(6.0, 900, 24.0)),
         0,
         1,
     ], streams=3, scale=0.7),
@@ -102,7 +102,7 @@ SINGLE = {
     "sink": model(32, 50, [layer(SINK, 4, 8, 4, 8, 16, 6, None)], streams=1),
     "gate": model(32, 50, [layer(GATE, 4, 8, 4, 8, 16, 6, None)], streams=1),
     "streams": model(32, 50, [layer(GATE, 1, 8, 4, 8, 16, 50, None), layer(SINK, 1, 8, 4, 8, 16, 50, dense(32))], streams=5),
-    "routed": model(32, 50, [layer(SINK, 1, 8, 4, 8, 16, 50, moe(24, 12, 3, groups=(3, 2), scale=2.0))], streams=1),
+    "routed": model(32, 50, [layer(SINK, 1, 8, 4, 8, 16, 50, moe(24, 15, 3, groups=(3, 2), scale=2.0))], streams=1),
     "shared_tensors": model(32, 50, [layer(SINK, 2, 8, 4, 8, 16, 5, dense(24)), 0, 0], streams=2),
 }
 
