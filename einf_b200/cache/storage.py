@@ -41,9 +41,8 @@ class CacheStorage:
         self._states: dict[int, torch.Tensor] = {}
         self.views: list[CacheView] = []
         for index, entry in enumerate(plan.entries):
-            if entry.owner != index:
-                continue
-            need, state = pages_of(entry.need), state_of(entry.need)
+            need = pages_of(entry.need) if entry.owner == index else None
+            state = state_of(entry.need) if entry.state_owner == index else None
             if need is not None and need.value_size == 0:
                 # the values are read out of the key rows: keys only
                 pages = self.pages_per_group[entry.group]
@@ -74,8 +73,9 @@ class CacheStorage:
                 kv = self._owned[entry.owner]
                 view = CacheView(group=entry.group, k=kv[0], v=kv[1], writes=entry.owner == index, page_size=page_size)
             if state_of(entry.need) is not None:
-                view.state = self._states[entry.owner]
-                view.writes = entry.owner == index
+                view.state = self._states[entry.state_owner]
+                if view.k is None:
+                    view.writes = entry.state_owner == index
             self.views.append(view)
 
     @property

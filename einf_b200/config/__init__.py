@@ -3,6 +3,7 @@ from .base import ConfigError, ModelConfig
 from .bomipel import BomipelConfig
 from .engine import EngineConfig
 from .kanavik import KanavikConfig
+from .pugadra import PugadraConfig
 from .qwen2 import Qwen2Config
 from .rekodra import RekodraConfig
 from .registry import (
@@ -22,6 +23,7 @@ register_architecture(BomipelConfig)
 register_architecture(KanavikConfig)
 register_architecture(RekodraConfig)
 register_architecture(SorizenConfig)
+register_architecture(PugadraConfig)
 
 __all__ = [
     "BomipelConfig",
@@ -32,6 +34,7 @@ __all__ = [
     "ModelConfig",
     "ModelSpec",
     "PartSpec",
+    "PugadraConfig",
     "Qwen2Config",
     "RekodraConfig",
     "ScheduleEntry",

@@ -19,7 +19,9 @@
 // With `keep_first` n > 0 a windowed token also sees the first n positions of its sequence
 // (j < n), at their true positions.  With `sink` (one float per query head) the softmax's
 // denominator of head h also holds exp(sink[h]): a column with no key and no value, unscaled.  With
-// `gate` (one float per token and query head) a head's mixed row is multiplied by it before it is rounded.
+// `gate` (one float per token and query head) a head's mixed row is multiplied by it before it is rounded; with
+// `value_gate` (one logit per element of the mixed heads, rows `value_gate_stride` apart) every element is
+// multiplied by the sigmoid of its own.
 // `value_stride` is the distance between two value rows in
 // elements: value_size for a cache of its own, the key size when the values are the leading
 // elements of the key rows (a latent cache that holds one row per token for both).
@@ -57,7 +59,8 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
                                T* __restrict__ out, int num_rows, int num_heads, int num_kv_heads,
                                int head_size, int value_size, int value_stride, int page_size, int num_pages,
                                int table_width, float scale, int window, int keep_first, int chunk, float softcap,
-                               const float* __restrict__ sink, const float* __restrict__ gate, int* status) {
+                               const float* __restrict__ sink, const float* __restrict__ gate,
+                               const T* __restrict__ value_gate, long long value_gate_stride, int* status) {
   __shared__ float q_smem[kWarpsPerBlock][kHeadLimit];
   pdl_launch_dependents();
   pdl_wait();
@@ -156,7 +159,11 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
 #pragma unroll
   for (int i = 0; i < kDimsPerLane; ++i) {
     const int d = lane + 32 * i;
-    if (d < value_size) o_row[d] = from_float<T>(acc[i] * inv);
+    if (d < value_size) {
+      float o = acc[i] * inv;
+      if (value_gate) o /= 1.f + expf(-to_float(value_gate[t * value_gate_stride + (long long)h * value_size + d]));
+      o_row[d] = from_float<T>(o);
+    }
   }
 }
 
@@ -379,7 +386,8 @@ extern "C" int einf_paged_attention_generic(const void* q, const void* k_cache, 
                                             int num_heads, int num_kv_heads, int head_size, int value_size,
                                             int value_stride, int page_size, int num_pages, int table_width,
                                             float scale, int window, int keep_first, int chunk, float softcap,
-                                            const float* sink, const float* gate, int* status, cudaStream_t stream) {
+                                            const float* sink, const float* gate, const void* value_gate,
+                                            long long value_gate_stride, int* status, cudaStream_t stream) {
   const int rows = num_tokens * num_heads;
   if (rows == 0) return 0;
   if (head_size > kMaxHeadSize || value_size > kMaxHeadSize || head_size <= 0 || value_size <= 0)
@@ -391,12 +399,12 @@ extern "C" int einf_paged_attention_generic(const void* q, const void* k_cache, 
       paged_attention_generic_kernel<T, 256><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
           (const T*)q, (const T*)k_cache, (const T*)v_cache, block_table, seq_of_token, positions, (T*)out,
           rows, num_heads, num_kv_heads, head_size, value_size, value_stride, page_size, num_pages, table_width,
-          scale, window, keep_first, chunk, softcap, sink, gate, status);
+          scale, window, keep_first, chunk, softcap, sink, gate, (const T*)value_gate, value_gate_stride, status);
     } else {
       paged_attention_generic_kernel<T, kMaxHeadSize><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
           (const T*)q, (const T*)k_cache, (const T*)v_cache, block_table, seq_of_token, positions, (T*)out,
           rows, num_heads, num_kv_heads, head_size, value_size, value_stride, page_size, num_pages, table_width,
-          scale, window, keep_first, chunk, softcap, sink, gate, status);
+          scale, window, keep_first, chunk, softcap, sink, gate, (const T*)value_gate, value_gate_stride, status);
     }
   })
   return (int)cudaGetLastError();

@@ -193,7 +193,12 @@ struct TcAttentionParams {
   float scale, softcap;     // scores are multiplied by scale; with a cap z they become z * tanh(score / z)
   const float* sink;        // [heads] or null: exp(sink[h]) joins the denominator of head h, with no key and no value
   const float* gate;        // [tokens, heads] or null: a head's mixed row is multiplied by it before it is rounded
+  const __nv_bfloat16* value_gate;   // rows of [heads * D] logits or null: every element is multiplied by the sigmoid of its own
+  long long value_gate_stride;       // elements from one token's logits to the next's
 };
+
+// What the division by the softmax's sum leaves, times the sigmoid of an output gate's logit.
+__device__ __forceinline__ float gate_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 
 __global__ void __launch_bounds__(kAttnThreads, 1)
 paged_prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -696,6 +701,23 @@ paged_prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q
       }
 #pragma unroll
       for (int c = 0; c < 32; ++c) v[c] = ((have ? v[c] : 0.f) * f_mine + take[c0 + c] * f_other) * inv;
+      if (p.value_gate && csize == 1 && ok && pos >= 0) {
+        const uint4* logits = reinterpret_cast<const uint4*>(p.value_gate + (size_t)(token0 + r) * p.value_gate_stride +
+                                                             head * D + g * kDimsHere + c0);
+        uint4 raw[4];
+#pragma unroll
+        for (int d = 0; d < 4; ++d) raw[d] = logits[d];
+#pragma unroll
+        for (int d = 0; d < 4; ++d) {
+          const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw[d]);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 z = __bfloat1622float2(h[e]);
+            v[8 * d + 2 * e] *= gate_sigmoid(z.x);
+            v[8 * d + 2 * e + 1] *= gate_sigmoid(z.y);
+          }
+        }
+      }
       if (csize > 1) {
 #pragma unroll
         for (int c = 0; c < 32; ++c) part_o[r * (D + 1) + g * kDimsHere + c0 + c] = v[c];
@@ -757,7 +779,12 @@ paged_prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q
       }
       __nv_bfloat16* dst = p.out + ((size_t)(token0 + row) * p.num_heads + head) * D;
 #pragma unroll
-      for (int j = 0; j < D / 32; ++j) dst[j * 32 + lane] = __float2bfloat16_rn(o[j] * inv);
+      for (int j = 0; j < D / 32; ++j) {
+        float v = o[j] * inv;
+        if (p.value_gate)
+          v *= gate_sigmoid(__bfloat162float(p.value_gate[(size_t)(token0 + row) * p.value_gate_stride + head * D + j * 32 + lane]));
+        dst[j * 32 + lane] = __float2bfloat16_rn(v);
+      }
     }
     cluster_leave();   // no CTA leaves while a peer may still read its shared memory
   }
@@ -818,6 +845,8 @@ struct TcDecodeParams {
   float scale, softcap;
   const float* sink;        // see TcAttentionParams
   const float* gate;        // see TcAttentionParams
+  const __nv_bfloat16* value_gate;
+  long long value_gate_stride;
   // A token's keys split over `splits` clusters, which meet in global memory: every cluster writes its
   // unnormalised share [16 heads][D + 2] (the accumulator, then maximum and sum) to split_out, every
   // CTA counts itself in split_count, and the CTA that finds itself the last adds the shares up.
@@ -1214,6 +1243,8 @@ paged_decode_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
     if (!kSplit) {
       if (p.sink && m != -INFINITY) l += exp2f(p.sink[first_head + row] * 1.4426950408889634f - m);
       if (p.gate) o *= p.gate[token_heads + first_head + row];
+      if (p.value_gate)
+        o *= gate_sigmoid(__bfloat162float(p.value_gate[(size_t)t * p.value_gate_stride + (first_head + row) * D + d]));
       p.out[(token_heads + first_head + row) * D + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     } else {
       float* share = p.split_out + (((size_t)pair * p.splits + split) * kDecHeads + row) * (D + 2);
@@ -1267,6 +1298,8 @@ paged_decode_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
       }
       if (p.sink && m != -INFINITY) l += exp2f(p.sink[first_head + row] * 1.4426950408889634f - m);
       if (p.gate) o *= p.gate[token_heads + first_head + row];
+      if (p.value_gate)
+        o *= gate_sigmoid(__bfloat162float(p.value_gate[(size_t)t * p.value_gate_stride + (first_head + row) * D + d]));
       p.out[(token_heads + first_head + row) * D + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     }
   }
@@ -1332,8 +1365,9 @@ extern "C" int einf_paged_prefill_attention_tcgen05(const void* q, const void* k
                                                     void* out, int num_tokens, int num_heads, int num_kv_heads,
                                                     int page_size, int num_pages, int table_width, float scale,
                                                     int window, int keep_first, int chunk, float softcap, int cluster,
-                                                    const float* sink, const float* gate, int* status,
-                                                    cudaStream_t stream) {
+                                                    const float* sink, const float* gate, const void* value_gate,
+                                                    long long value_gate_stride, int* status, cudaStream_t stream) {
+  if (((uintptr_t)value_gate | (uintptr_t)(value_gate_stride * 2)) % 16) return (int)cudaErrorInvalidValue;
   if (num_tiles == 0) return 0;
   if (cluster < 1 || cluster > 8) return (int)cudaErrorInvalidValue;
   if (keep_first < 0 || (keep_first > 0 && window > 0 && cluster != 1)) return (int)cudaErrorInvalidValue;
@@ -1368,6 +1402,8 @@ extern "C" int einf_paged_prefill_attention_tcgen05(const void* q, const void* k
   p.softcap = softcap;
   p.sink = sink;
   p.gate = gate;
+  p.value_gate = (const __nv_bfloat16*)value_gate;
+  p.value_gate_stride = value_gate_stride;
   cudaError_t e = cudaFuncSetAttribute(paged_prefill_attention_tcgen05_kernel,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
   if (e != cudaSuccess) return (int)e;
@@ -1436,7 +1472,8 @@ extern "C" int einf_paged_decode_attention_tcgen05(const void* q, const void* k_
                                                    int num_pages, int table_width, float scale, int window,
                                                    int keep_first, int chunk, float softcap, int cluster, int splits,
                                                    float* split_out, int* split_count, const float* sink, const float* gate,
-                                                   int* status, cudaStream_t stream) {
+                                                   const void* value_gate, long long value_gate_stride, int* status,
+                                                   cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (cluster < 1 || cluster > kDecMaxCluster) return (int)cudaErrorInvalidValue;
   if (splits < 1 || splits > kDecMaxSplits || (splits > 1 && (!split_out || !split_count))) return (int)cudaErrorInvalidValue;
@@ -1472,6 +1509,8 @@ extern "C" int einf_paged_decode_attention_tcgen05(const void* q, const void* k_
   p.softcap = softcap;
   p.sink = sink;
   p.gate = gate;
+  p.value_gate = (const __nv_bfloat16*)value_gate;
+  p.value_gate_stride = value_gate_stride;
   p.splits = splits;
   p.split_out = split_out;
   p.split_count = split_count;

@@ -818,10 +818,26 @@ __global__ void activation_bf16x8_kernel(const __nv_bfloat16* __restrict__ x, __
 // feed-forward with another gate than SiLU.  The dense bfloat16 form computes the GELU's tanh as
 // 1 - 2 / (exp(2 a) + 1) with the hardware exponential and reciprocal (the result is rounded to
 // bfloat16); the generic form, which the 32-bit path uses, calls tanhf.
+// Kind 5 clamps both branches, g = min(gate, limit) and u = clamp(up, -limit, limit), and gives
+// g sigmoid(slope g) (u + shift).
 // ---------------------------------------------------------------------------
+struct GateJoin {
+  int kind;
+  float limit, slope, shift;
+};
+
+__device__ __forceinline__ float join_branches(float g, float u, const GateJoin& join) {
+  if (join.kind == 5) {
+    g = fminf(g, join.limit);
+    u = fminf(fmaxf(u, -join.limit), join.limit);
+    return g / (1.f + expf(-join.slope * g)) * (u + join.shift);
+  }
+  return activate(g, join.kind) * u;
+}
+
 template <typename TIn, typename T>
 __global__ void act_mul_kernel(const TIn* __restrict__ gate_up, int splits, size_t split_stride, T* __restrict__ out,
-                               int intermediate, int kind, size_t total) {
+                               int intermediate, const GateJoin join, size_t total) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -830,7 +846,7 @@ __global__ void act_mul_kernel(const TIn* __restrict__ gate_up, int splits, size
     const int i = (int)(idx - t * intermediate);
     const float g = sum_splits(gate_up + t * 2 * intermediate + i, splits, split_stride);
     const float u = sum_splits(gate_up + t * 2 * intermediate + intermediate + i, splits, split_stride);
-    out[idx] = from_float<T>(activate(g, kind) * u);
+    out[idx] = from_float<T>(join_branches(g, u, join));
   }
 }
 
@@ -844,8 +860,17 @@ __device__ __forceinline__ float activate_fast(float z, int kind) {
   return activate(z, kind);
 }
 
+__device__ __forceinline__ float join_branches_fast(float g, float u, const GateJoin& join) {
+  if (join.kind == 5) {
+    g = fminf(g, join.limit);
+    u = fminf(fmaxf(u, -join.limit), join.limit);
+    return __fdividef(g, 1.f + __expf(-join.slope * g)) * (u + join.shift);
+  }
+  return activate_fast(g, join.kind) * u;
+}
+
 __global__ void act_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gate_up, __nv_bfloat16* __restrict__ out,
-                                      int intermediate, int chunks_per_row, int kind) {
+                                      int intermediate, int chunks_per_row, const GateJoin join) {
   pdl_launch_dependents();
   pdl_wait();
   const unsigned t = blockIdx.x / (unsigned)chunks_per_row;
@@ -863,7 +888,7 @@ __global__ void act_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gate_up,
     for (int e = 0; e < 4; ++e) {
       const float2 gf = __bfloat1622float2(gp[e]);
       const float2 uf = __bfloat1622float2(up[e]);
-      rp[e] = __floats2bfloat162_rn(activate_fast(gf.x, kind) * uf.x, activate_fast(gf.y, kind) * uf.y);
+      rp[e] = __floats2bfloat162_rn(join_branches_fast(gf.x, uf.x, join), join_branches_fast(gf.y, uf.y, join));
     }
     *reinterpret_cast<uint4*>(out + (size_t)t * intermediate + i) = result;
   }
@@ -1563,7 +1588,9 @@ extern "C" int einf_silu_mul(const void* gate_up, int in_dtype, int splits, long
 }
 
 extern "C" int einf_act_mul(const void* gate_up, int in_dtype, int splits, long long split_stride, void* out,
-                            int dtype, long long num_tokens, int intermediate, int kind, cudaStream_t stream) {
+                            int dtype, long long num_tokens, int intermediate, int kind, float limit, float slope,
+                            float shift, cudaStream_t stream) {
+  const GateJoin join{kind, limit, slope, shift};
   const size_t total = (size_t)num_tokens * intermediate;
   if (total == 0) return 0;
   const int threads = 256;
@@ -1573,14 +1600,14 @@ extern "C" int einf_act_mul(const void* gate_up, int in_dtype, int splits, long 
     const int chunks = (vectors_per_row + threads - 1) / threads;
     if ((long long)chunks * num_tokens < (1ll << 31))
       return (int)launch_pdl(act_mul_bf16x8_kernel, (int)(chunks * num_tokens), threads, 0, stream,
-                             (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, intermediate, chunks, kind);
+                             (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, intermediate, chunks, join);
   }
   size_t blocks = (total + threads - 1) / threads;
   if (blocks > 148 * 16) blocks = 148 * 16;
   EINF_DISPATCH_2(in_dtype, TIn, {
     EINF_DISPATCH_2(dtype, T, {
       return (int)launch_pdl(act_mul_kernel<TIn, T>, (int)blocks, threads, 0, stream, (const TIn*)gate_up, splits,
-                             (size_t)split_stride, (T*)out, intermediate, kind, total);
+                             (size_t)split_stride, (T*)out, intermediate, join, total);
     })
   })
 }

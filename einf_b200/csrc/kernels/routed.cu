@@ -1,7 +1,8 @@
 // A routed feed-forward (mixture of experts) in five steps, all on the device so that a step
 // never waits for the host to learn how many tokens an expert got:
 //
-//   einf_router_topk   per token: the `top_k` largest router logits (ties to the lower index),
+//   einf_router_topk   per token: the `top_k` largest router logits, a stored bias added first if
+//                      there is one (ties to the lower index),
 //                      their weights sigmoid(z) or softmax(z) over all experts, optionally
 //                      divided by their sum (plus a constant) and multiplied by another; 32-bit throughout.  With a correction the choice goes
 //                      by score + correction (the weights stay the scores); with groups only the
@@ -34,8 +35,8 @@ constexpr int kMaxExpertsPerLane = 32;   // experts up to 1024
 
 __global__ void router_topk_kernel(const float* __restrict__ logits, int splits, size_t split_stride, int num_tokens,
                                    int row_width, int num_experts, int top_k, int score, int renormalise,
-                                   float renormalise_eps, float weight_scale, const float* __restrict__ correction,
-                                   int group_count, int group_keep, int group_best, int* __restrict__ expert_ids,
+                                   float renormalise_eps, float weight_scale, const float* __restrict__ bias,
+                                   const float* __restrict__ correction, int group_count, int group_keep, int group_best, int* __restrict__ expert_ids,
                                    float* __restrict__ weights) {
   // per warp of the CTA: [num_experts] what the choice goes by | [num_experts] the scores (with a correction) |
   // [group_count] 1 for a group that may be chosen from
@@ -52,7 +53,7 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int splits,
   for (int e = lane; e < num_experts; e += 32) {
     float v = 0.f;
     for (int s = 0; s < splits; ++s) v += logits[(size_t)s * split_stride + (size_t)t * row_width + e];
-    z[e] = v;
+    z[e] = bias ? v + bias[e] : v;
   }
   __syncwarp();
   float z_max = -INFINITY;
@@ -428,8 +429,9 @@ using namespace einf;
 
 extern "C" int einf_router_topk(const float* logits, int splits, long long split_stride, int num_tokens,
                                 int row_width, int num_experts, int top_k, int score, int renormalise,
-                                float renormalise_eps, float weight_scale, const float* correction, int group_count,
-                                int group_keep, int group_best, int* expert_ids, float* weights, cudaStream_t stream) {
+                                float renormalise_eps, float weight_scale, const float* bias, const float* correction,
+                                int group_count, int group_keep, int group_best, int* expert_ids, float* weights,
+                                cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (num_experts <= 0 || num_experts > 32 * kMaxExpertsPerLane || top_k <= 0 || top_k > num_experts ||
       row_width < num_experts)
@@ -442,7 +444,7 @@ extern "C" int einf_router_topk(const float* logits, int splits, long long split
   const size_t per_warp = (size_t)(correction ? 2 : 1) * num_experts + group_count;
   return (int)launch_pdl(router_topk_kernel, blocks, threads, (size_t)(threads / 32) * per_warp * sizeof(float), stream,
                          logits, splits < 1 ? 1 : splits, (size_t)split_stride, num_tokens, row_width, num_experts, top_k,
-                         score, renormalise, renormalise_eps, weight_scale, correction, group_count, group_keep,
+                         score, renormalise, renormalise_eps, weight_scale, bias, correction, group_count, group_keep,
                          group_best, expert_ids, weights);
 }
 

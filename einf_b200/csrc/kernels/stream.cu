@@ -1,6 +1,7 @@
 // The residual stream between sublayers, for blocks that do more to it than add and normalise:
 //   - a residual multiplier on every sublayer's output,
 //   - a short causal convolution over time in front of a sublayer, in the launch of the norm,
+//   - a norm behind a sublayer, of its output before that is added to the stream,
 //   - a per-layer token input after the feed-forward,
 //   - a weighted sum over the results of all layers so far in place of the layer's own result.
 // The stream is 32-bit; pending sublayer outputs arrive as up to two terms, each a [T, H] matrix
@@ -187,8 +188,174 @@ __global__ void conv_rows_state_kernel(const float* __restrict__ h, float* __res
 }
 
 // ---------------------------------------------------------------------------
+// What a sublayer leaves goes into the stream and the next one's input comes out of it, in one pass:
+//   y = pending[t];  post != null: y = y * rsqrt(mean(y^2) + post_eps) * post
+//   residual[t] += scale * y
+//   out[t] = residual[t] * rsqrt(mean(residual[t]^2) + eps) * weight   (weight null: residual[t] itself; out null: nothing)
+// A team of kTeam threads has a row, kVec groups of four columns a thread, in registers between the two
+// sums of squares: a warp (eight rows a CTA) for many rows, a CTA for few or wide ones.  Loads come
+// first, without a branch between them (an index past the row is clamped, its value unused), so that
+// a whole row is in flight at once.
+// ---------------------------------------------------------------------------
+// kBatch: partial sums of which all loads are in flight at once (they sit in L2); 1: there are none
+template <int kBatch>
+__device__ __forceinline__ float4 pending4(const void* p, int dtype, int splits, long long stride, size_t idx) {
+  if (dtype == kBFloat16) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < (kBatch == 1 ? 1 : splits); ++s) {
+      const uint2 raw = *(const uint2*)((const __nv_bfloat16*)p + (size_t)s * stride + idx);
+      const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&raw.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&raw.y);
+      v.x += a.x; v.y += a.y; v.z += b.x; v.w += b.y;
+    }
+    return v;
+  }
+  const float* q = (const float*)p + idx;
+  if (kBatch == 1 || splits == 1) return *(const float4*)q;
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int s0 = 0; s0 < splits; s0 += kBatch) {
+    float4 part[kBatch];
+#pragma unroll
+    for (int e = 0; e < kBatch; ++e) part[e] = *(const float4*)(q + (size_t)min(s0 + e, splits - 1) * stride);
+#pragma unroll
+    for (int e = 0; e < kBatch; ++e)
+      if (s0 + e < splits) { v.x += part[e].x; v.y += part[e].y; v.z += part[e].z; v.w += part[e].w; }
+  }
+  return v;
+}
+
+__device__ __forceinline__ void store_row4(float* p, const float4& v) { *(float4*)p = v; }
+__device__ __forceinline__ void store_row4(__nv_bfloat16* p, const float4& v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 raw;
+  raw.x = *(const uint32_t*)&a;
+  raw.y = *(const uint32_t*)&b;
+  *(uint2*)p = raw;
+}
+
+template <typename TOut, int kTeam, int kVec>
+__global__ void stream_norm_kernel(const __grid_constant__ Pending pending, float scale, const float* __restrict__ post,
+                                   float post_eps, float* __restrict__ residual, const float* __restrict__ weight,
+                                   float eps, TOut* __restrict__ out, int hidden, int num_rows) {
+  __shared__ float red[33];
+  pdl_launch_dependents();
+  const int row = kTeam == 32 ? (int)((blockIdx.x * blockDim.x + threadIdx.x) >> 5) : (int)blockIdx.x;
+  const int member = kTeam == 32 ? (int)(threadIdx.x & 31) : (int)threadIdx.x;
+  const size_t base = (size_t)row * hidden;
+  pdl_wait();
+  if (kTeam == 32 && row >= num_rows) return;
+  auto team_sum = [&](float v) { return kTeam == 32 ? warp_sum(v) : block_sum(v, red); };
+  auto column = [&](int j) { return (j * kTeam + member) * 4; };
+  const bool adds = pending.a != nullptr;
+  constexpr int kBatch = kTeam == 32 ? 1 : 16 / kVec;
+  float4 x[kVec];
+#pragma unroll
+  for (int j = 0; j < kVec; ++j) x[j] = *(const float4*)(residual + base + min(column(j), hidden - 4));
+  if (adds) {
+    float4 y[kVec];
+#pragma unroll
+    for (int j = 0; j < kVec; ++j)
+      y[j] = pending4<kBatch>(pending.a, pending.a_dtype, pending.a_splits, pending.a_stride, base + min(column(j), hidden - 4));
+    if (post) {
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < kVec; ++j)
+        if (column(j) < hidden) ss += y[j].x * y[j].x + y[j].y * y[j].y + y[j].z * y[j].z + y[j].w * y[j].w;
+      const float inv = rsqrtf(team_sum(ss) / (float)hidden + post_eps);
+#pragma unroll
+      for (int j = 0; j < kVec; ++j) {
+        const float4 w = *(const float4*)(post + min(column(j), hidden - 4));
+        y[j].x *= inv * w.x; y[j].y *= inv * w.y; y[j].z *= inv * w.z; y[j].w *= inv * w.w;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+      x[j].x = fmaf(scale, y[j].x, x[j].x); x[j].y = fmaf(scale, y[j].y, x[j].y);
+      x[j].z = fmaf(scale, y[j].z, x[j].z); x[j].w = fmaf(scale, y[j].w, x[j].w);
+      if (column(j) < hidden) *(float4*)(residual + base + column(j)) = x[j];
+    }
+  }
+  if (!out) return;
+  float inv = 1.f;
+  if (weight) {
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < kVec; ++j)
+      if (column(j) < hidden) ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
+    inv = rsqrtf(team_sum(ss) / (float)hidden + eps);
+  }
+#pragma unroll
+  for (int j = 0; j < kVec; ++j) {
+    if (column(j) >= hidden) continue;
+    float4 v = x[j];
+    if (weight) {
+      const float4 w = *(const float4*)(weight + column(j));
+      v.x *= inv * w.x; v.y *= inv * w.y; v.z *= inv * w.z; v.w *= inv * w.w;
+    }
+    store_row4(out + base + column(j), v);
+  }
+}
+
+// The same for two pending terms, and for widths that are no multiple of four or too wide for registers: one CTA
+// per row, in shared memory.
+template <typename TOut>
+__global__ void stream_norm_any_kernel(const __grid_constant__ Pending pending, float scale, const float* __restrict__ post,
+                                       float post_eps, float* __restrict__ residual, const float* __restrict__ weight,
+                                       float eps, TOut* __restrict__ out, int hidden) {
+  extern __shared__ float smem[];
+  float* row = smem;
+  float* red = smem + hidden;
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t base = (size_t)blockIdx.x * hidden;
+  const bool adds = pending.a != nullptr || pending.b != nullptr;
+  // every thread reads back the columns it wrote itself
+  float factor = 1.f;
+  if (adds) {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+      row[c] = pending_sum(pending, base + c);
+      ss = fmaf(row[c], row[c], ss);
+    }
+    if (post) factor = rsqrtf(block_sum(ss, red) / (float)hidden + post_eps);
+  }
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    float v = residual[base + c];
+    if (adds) {
+      v = fmaf(scale, post ? row[c] * (factor * post[c]) : row[c], v);
+      residual[base + c] = v;
+    }
+    row[c] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (!out) return;
+  const float inv = weight ? rsqrtf(block_sum(ss, red) / (float)hidden + eps) : 1.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x)
+    out[base + c] = from_float<TOut>(weight ? row[c] * (inv * weight[c]) : row[c]);
+}
+
+// out[t, d] = gelu(sum_s product[s][t, d]) * table[token[t], d]
+template <typename TIn, typename TW, typename TOut>
+__global__ void side_gate_kernel(const TIn* __restrict__ product, int splits, long long split_stride,
+                                 const TW* __restrict__ table, const int* __restrict__ token_ids, TOut* __restrict__ out,
+                                 int num_tokens, int side, int vocab) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long total = (long long)num_tokens * side;
+  for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
+       idx += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(idx / side), d = (int)(idx - (long long)t * side);
+    int token = token_ids[t];
+    token = token < 0 ? 0 : (token >= vocab ? vocab - 1 : token);     // a bad id was reported by the embedding
+    float s = 0.f;
+    for (int k = 0; k < splits; ++k) s += to_float(product[(size_t)k * split_stride + idx]);
+    out[idx] = from_float<TOut>(gelu_tanh_f(s) * to_float(table[(size_t)token * side + d]));
+  }
+}
+
+// ---------------------------------------------------------------------------
 // The end of a layer.  One CTA per token, the row x in shared memory:
-//   x = residual[t] + scale * pending[t]
+//   x = residual[t] + scale * pending[t]   (post != null: of its RMS norm, as above)
 //   token input (table != null):  s = gate x  [n];  g = gelu(s) * table[token]  [n];  y = proj_t^T g  [H];
 //                                 x += scale * y * rsqrt(mean(y^2) + eps) * norm
 //   depth average (history != null):  history[index + 1][t] = x;
@@ -203,7 +370,7 @@ __global__ void stream_tail_kernel(float* __restrict__ residual, const __grid_co
                                    const TW* __restrict__ gate, const TW* __restrict__ proj_t,
                                    const float* __restrict__ norm, int side, int vocab, float eps,
                                    float* __restrict__ history, int depth_index, const float* __restrict__ depth_weight,
-                                   long long history_stride, int hidden) {
+                                   long long history_stride, const float* __restrict__ post, float post_eps, int hidden) {
   extern __shared__ float smem[];
   float* x = smem;                   // [hidden]
   float* y = x + hidden;             // [hidden]
@@ -214,10 +381,21 @@ __global__ void stream_tail_kernel(float* __restrict__ residual, const __grid_co
   const int t = blockIdx.x;
   const size_t base = (size_t)t * hidden;
   const bool adds = pending.a != nullptr || pending.b != nullptr;
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-    float v = residual[base + c];
-    if (adds) v += scale * pending_sum(pending, base + c);
-    x[c] = v;
+  if (post && adds) {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+      const float v = pending_sum(pending, base + c);
+      y[c] = v;
+      ss = fmaf(v, v, ss);
+    }
+    const float factor = scale * rsqrtf(block_sum(ss, red) / (float)hidden + post_eps);
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) x[c] = fmaf(factor * post[c], y[c], residual[base + c]);
+  } else {
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+      float v = residual[base + c];
+      if (adds) v += scale * pending_sum(pending, base + c);
+      x[c] = v;
+    }
   }
   __syncthreads();
   if (table) {
@@ -295,7 +473,8 @@ stream_tail_tokens_kernel(float* __restrict__ residual, const __grid_constant__ 
                           const int* __restrict__ token_ids, const TW* __restrict__ table, const TW* __restrict__ gate,
                           const TW* __restrict__ proj_t, const float* __restrict__ norm, int side, int vocab, float eps,
                           float* __restrict__ history, int depth_index, const float* __restrict__ depth_weight,
-                          long long history_stride, int hidden, int num_tokens) {
+                          long long history_stride, const float* __restrict__ post, float post_eps, int hidden,
+                          int num_tokens) {
   extern __shared__ float4 smem4[];
   float* x = (float*)smem4;          // [TB, hidden]
   float* y = x + TB * hidden;        // [TB, hidden]
@@ -308,15 +487,40 @@ stream_tail_tokens_kernel(float* __restrict__ residual, const __grid_constant__ 
   const int t0 = blockIdx.x * TB;
   const int count = min(TB, num_tokens - t0);
   const bool adds = pending.a != nullptr || pending.b != nullptr;
-  for (int idx = tid; idx < TB * hidden; idx += kTailThreads) {
-    const int i = idx / hidden;
-    float v = 0.f;
-    if (i < count) {
-      const size_t at = (size_t)t0 * hidden + idx;
-      v = residual[at];
-      if (adds) v += scale * pending_sum(pending, at);
+  if (post && adds) {
+    // the pending rows and their sums of squares first; every thread reads back the columns it wrote itself
+#pragma unroll 1
+    for (int i = 0; i < TB; ++i) {
+      float ss = 0.f;
+      for (int c = tid; c < hidden; c += kTailThreads) {
+        const float v = i < count ? pending_sum(pending, (size_t)(t0 + i) * hidden + c) : 0.f;
+        y[i * hidden + c] = v;
+        ss = fmaf(v, v, ss);
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) red[i * kWarps + warp] = ss;
     }
-    x[idx] = v;
+    __syncthreads();
+#pragma unroll 1
+    for (int i = 0; i < TB; ++i) {
+      float total = 0.f;
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) total += red[i * kWarps + w];
+      const float factor = scale * rsqrtf(total / (float)hidden + post_eps);
+      for (int c = tid; c < hidden; c += kTailThreads)
+        x[i * hidden + c] = i < count ? fmaf(factor * post[c], y[i * hidden + c], residual[(size_t)(t0 + i) * hidden + c]) : 0.f;
+    }
+  } else {
+    for (int idx = tid; idx < TB * hidden; idx += kTailThreads) {
+      const int i = idx / hidden;
+      float v = 0.f;
+      if (i < count) {
+        const size_t at = (size_t)t0 * hidden + idx;
+        v = residual[at];
+        if (adds) v += scale * pending_sum(pending, at);
+      }
+      x[idx] = v;
+    }
   }
   __syncthreads();
   if (table) {
@@ -489,12 +693,71 @@ extern "C" int einf_norm_conv(const void* pend_a, int a_dtype, int a_splits, lon
   })
 }
 
+extern "C" int einf_stream_norm(const void* pend_a, int a_dtype, int a_splits, long long a_stride, const void* pend_b,
+                                int b_dtype, int b_splits, long long b_stride, float scale, const float* post,
+                                float post_eps, float* residual, const float* weight, float eps, void* out, int out_dtype,
+                                int num_tokens, int hidden, cudaStream_t stream) {
+  if (num_tokens == 0) return 0;
+  if (hidden <= 0) return (int)cudaErrorInvalidValue;
+  const Pending pending{pend_a, a_dtype, a_splits, a_stride, pend_b, b_dtype, b_splits, b_stride};
+  // four columns an access: 16 bytes of floats, 8 of bfloat16
+  auto pieces = [](const void* p, int dtype, int splits, long long stride) {
+    return (uintptr_t)p % (dtype == kBFloat16 ? 8 : 16) == 0 && (splits <= 1 || stride % 4 == 0);
+  };
+  const bool vectors = hidden % 4 == 0 && hidden <= 8192 && !pend_b && pieces(pend_a, a_dtype, a_splits, a_stride) &&
+                       pieces(residual, kFloat32, 1, 0) &&
+                       pieces(post, kFloat32, 1, 0) && pieces(weight, kFloat32, 1, 0) && pieces(out, out_dtype, 1, 0);
+#define EINF_STREAM_NORM(TEAM, VEC, GRID, THREADS)                                                                      \
+  return (int)launch_pdl(stream_norm_kernel<T, TEAM, VEC>, GRID, THREADS, 0, stream, pending, scale, post, post_eps,    \
+                         residual, weight, eps, (T*)out, hidden, num_tokens)
+  EINF_DISPATCH_2(out_dtype, T, {
+    if (vectors) {
+      // partial sums want every load of a row in flight: a warp a row only where there are none
+      if (num_tokens >= 256 && hidden <= 2048 && a_splits <= 1) {
+        const int grid = (num_tokens + 7) / 8;
+        if (hidden <= 1024) EINF_STREAM_NORM(32, 8, grid, 256);
+        EINF_STREAM_NORM(32, 16, grid, 256);
+      }
+      if (hidden <= 512) EINF_STREAM_NORM(128, 1, num_tokens, 128);
+      if (hidden <= 1024) EINF_STREAM_NORM(256, 1, num_tokens, 256);
+      if (hidden <= 2048) EINF_STREAM_NORM(512, 1, num_tokens, 512);
+      EINF_STREAM_NORM(512, 4, num_tokens, 512);
+    }
+    const size_t smem = (size_t)(hidden + 33) * sizeof(float);
+    if (smem > 48 * 1024) {
+      cudaError_t e = cudaFuncSetAttribute(stream_norm_any_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return (int)e;
+    }
+    return (int)launch_pdl(stream_norm_any_kernel<T>, num_tokens, row_threads(hidden), smem, stream, pending, scale, post,
+                           post_eps, residual, weight, eps, (T*)out, hidden);
+  })
+#undef EINF_STREAM_NORM
+}
+
+extern "C" int einf_side_gate(const void* product, int in_dtype, int splits, long long split_stride, const void* table,
+                              int table_dtype, const int* token_ids, void* out, int out_dtype, int num_tokens, int side,
+                              int vocab, cudaStream_t stream) {
+  if (num_tokens == 0 || side <= 0) return side < 0 ? (int)cudaErrorInvalidValue : 0;
+  const long long total = (long long)num_tokens * side;
+  long long blocks = (total + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  EINF_DISPATCH_2(in_dtype, TIn, {
+    EINF_DISPATCH_2(table_dtype, TW, {
+      EINF_DISPATCH_2(out_dtype, TOut, {
+        return (int)launch_pdl(side_gate_kernel<TIn, TW, TOut>, (int)blocks, 256, 0, stream, (const TIn*)product,
+                               splits < 1 ? 1 : splits, split_stride, (const TW*)table, token_ids, (TOut*)out, num_tokens,
+                               side, vocab);
+      })
+    })
+  })
+}
+
 extern "C" int einf_stream_tail(float* residual, const void* pend_a, int a_dtype, int a_splits, long long a_stride,
                                 const void* pend_b, int b_dtype, int b_splits, long long b_stride, float scale,
                                 const int* token_ids, const void* table, const void* gate, const void* proj_t,
                                 int weight_dtype, const float* norm, int side, int vocab, float eps, float* history,
-                                int depth_index, const float* depth_weight, long long history_stride, int num_tokens,
-                                int hidden, cudaStream_t stream) {
+                                int depth_index, const float* depth_weight, long long history_stride,
+                                const float* post, float post_eps, int num_tokens, int hidden, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (hidden <= 0 || side < 0) return (int)cudaErrorInvalidValue;
   const Pending pending{pend_a, a_dtype, a_splits, a_stride, pend_b, b_dtype, b_splits, b_stride};
@@ -514,7 +777,7 @@ extern "C" int einf_stream_tail(float* residual, const void* pend_a, int a_dtype
     }                                                                                                                   \
     return (int)launch_pdl(kernel, blocks, kTailThreads, bytes(TB), stream, residual, pending, scale, token_ids,       \
                            (const T*)table, (const T*)gate, (const T*)proj_t, norm, side, vocab, eps, history,          \
-                           depth_index, depth_weight, history_stride, hidden, num_tokens);                              \
+                               depth_index, depth_weight, history_stride, post, post_eps, hidden, num_tokens);              \
   })
       if (each == 8) EINF_TAIL(8)
       if (each == 1) EINF_TAIL(1)
@@ -531,6 +794,6 @@ extern "C" int einf_stream_tail(float* residual, const void* pend_a, int a_dtype
     }
     return (int)launch_pdl(stream_tail_kernel<T>, num_tokens, threads, smem, stream, residual, pending, scale,
                            token_ids, (const T*)table, (const T*)gate, (const T*)proj_t, norm, side, vocab, eps,
-                           history, depth_index, depth_weight, history_stride, hidden);
+                           history, depth_index, depth_weight, history_stride, post, post_eps, hidden);
   })
 }

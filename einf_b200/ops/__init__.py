@@ -319,20 +319,24 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
 
 
 #: activations of a gated feed-forward's gate branch (``silu`` has launches of its own, :func:`silu_mul`)
-GATE_ACTIVATIONS = {"silu": 2, "gelu_tanh": 1}
+GATE_ACTIVATIONS = {"silu": 2, "gelu_tanh": 1, "clamped_swish": 5}
 
 
-def act_mul(gate_up: torch.Tensor, out: torch.Tensor, kind: str) -> None:
+def act_mul(gate_up: torch.Tensor, out: torch.Tensor, kind: str, limit: float = 0.0, slope: float = 1.0,
+            up_shift: float = 0.0) -> None:
     """``out = act(gate_up[:, :I]) * gate_up[:, I:]`` with ``act`` one of :data:`GATE_ACTIVATIONS`;
-    ``gate_up`` may be float32 partial sums ``[splits, tokens, 2 I]`` of a split-K product."""
+    ``gate_up`` may be float32 partial sums ``[splits, tokens, 2 I]`` of a split-K product.  ``clamped_swish``
+    clamps both branches, ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``, and gives
+    ``g sigmoid(slope g) (u + up_shift)``; the three constants are its alone."""
     tokens, inter = out.shape
     splits, stride = _maybe_split(gate_up, tokens, 2 * inter, "gate_up")
     if kind not in GATE_ACTIVATIONS:
         raise ValueError(f"unknown gate activation {kind!r}; known: {sorted(GATE_ACTIVATIONS)}")
-    fn = _fn("einf_act_mul", [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p])
+    fn = _fn("einf_act_mul", [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_longlong, c_int, c_int, c_float,
+                              c_float, c_float, c_void_p])
     _check(
         fn(_dev(gate_up, "gate_up"), _code(gate_up), splits, stride, _dev(out, "out"), _code(out), tokens, inter,
-           GATE_ACTIVATIONS[kind], _stream()),
+           GATE_ACTIVATIONS[kind], float(limit), float(slope), float(up_shift), _stream()),
         "act_mul",
     )
 
@@ -526,6 +530,23 @@ def project(
     return out
 
 
+def _value_gate(value_gate: Optional[torch.Tensor], q: torch.Tensor, value_size: int, aligned: bool) -> tuple[int, int]:
+    """Pointer and row stride of the logits of an output gate, one per element of the mixed heads:
+    ``[tokens, heads * value_size]`` of q's dtype, rows contiguous (columns of a wider matrix are fine);
+    ``aligned``: the kernel reads them in 16-byte pieces."""
+    if value_gate is None:
+        return 0, 0
+    if value_gate.dtype != q.dtype or value_gate.shape != (q.shape[0], q.shape[1] * value_size) or \
+            value_gate.stride(1) != 1:
+        raise ValueError(f"value_gate must be {q.dtype} {(q.shape[0], q.shape[1] * value_size)} with contiguous rows")
+    if not value_gate.is_cuda:
+        raise KernelError("value_gate must be on a CUDA device: there is no CPU path")
+    size = value_gate.element_size()
+    if aligned and (value_gate.data_ptr() % 16 or value_gate.stride(0) * size % 16):
+        raise UnsupportedSize("value_gate rows must start on 16-byte boundaries")
+    return value_gate.data_ptr(), value_gate.stride(0)
+
+
 def _check_gate(gate: Optional[torch.Tensor], tokens: int, heads: int) -> None:
     if gate is not None and (gate.dtype != torch.float32 or gate.shape != (tokens, heads)):
         raise ValueError(f"gate must be float32 {(tokens, heads)}, got {gate.dtype} {tuple(gate.shape)}")
@@ -548,6 +569,7 @@ def paged_attention_generic(
     values_in_keys: Optional[int] = None,
     sink: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None,
+    value_gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Causal attention of every token of the batch over the pages of its request.
 
@@ -561,7 +583,8 @@ def paged_attention_generic(
     token's value is the first n elements of its key row (one cached row serves as both).
     ``sink`` (float32 ``[heads]``): the softmax's denominator of head h also holds ``exp(sink[h])``,
     unscaled, with no key and no value.  ``gate`` (float32 ``[tokens, heads]``): a head's mixed row is multiplied
-    by it before it is rounded.
+    by it before it is rounded.  ``value_gate`` (q's dtype, ``[tokens, heads * value_size]``, rows may be columns of
+    a wider matrix): every element of the mixed heads is multiplied by the sigmoid of its own logit.
     """
     tokens, num_heads, head_size = q.shape
     if sink is not None and (sink.dtype != torch.float32 or sink.shape != (num_heads,)):
@@ -591,7 +614,7 @@ def paged_attention_generic(
         "einf_paged_attention_generic",
         [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
          c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
-         c_void_p],
+         c_longlong, c_void_p, c_void_p],
     )
     _check(
         fn(_dev(q, "q"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), _code(q),
@@ -600,7 +623,7 @@ def paged_attention_generic(
            head_size, value_size, value_stride, page_size, num_pages, block_table.shape[1], float(scale),
            int(window) if window else 0, int(keep_first) if window else 0, int(chunk) if chunk else 0,
            float(softcap) if softcap else 0.0, _opt(sink, "sink", torch.float32), _opt(gate, "gate", torch.float32),
-           _dev(status, "status"), _stream()),
+           *_value_gate(value_gate, q, value_size, False), _dev(status, "status"), _stream()),
         "paged_attention_generic",
     )
 
@@ -900,6 +923,117 @@ def qkv_norm_store(
     )
 
 
+def gate_in_place(qkv: torch.Tensor, channels: int, dtype: torch.dtype) -> bool:
+    """Whether the attention kernels can read an output gate's logits as the columns from ``channels`` on of
+    the product ``qkv`` (no partial sums, the activation type, rows on 16-byte boundaries)."""
+    return (qkv.dim() == 2 and qkv.dtype == dtype and qkv.is_contiguous()
+            and channels * qkv.element_size() % 16 == 0 and qkv.shape[1] * qkv.element_size() % 16 == 0)
+
+
+def qkv_conv_store(
+    qkv: torch.Tensor,
+    bias: Optional[torch.Tensor],
+    conv_weight: Optional[torch.Tensor],
+    conv_state: Optional[torch.Tensor],
+    seq_of_token: torch.Tensor,
+    q_start: torch.Tensor,
+    state_slots: torch.Tensor,
+    slots: Optional[torch.Tensor],
+    q_out: torch.Tensor,
+    k_cache: Optional[torch.Tensor],
+    v_cache: Optional[torch.Tensor],
+    num_heads: int,
+    num_kv_heads: int,
+    key_size: int,
+    value_size: int,
+    status: torch.Tensor,
+    positions: Optional[torch.Tensor] = None,
+    inv_freq: Optional[torch.Tensor] = None,
+    interleaved: bool = False,
+    gate_out: Optional[torch.Tensor] = None,
+    single_tokens: bool = False,
+) -> None:
+    """Bias, a causal convolution over time on every channel, rotation and cache write.
+
+    A row of ``qkv`` (or of its float32 split-K partial sums) is ``[heads * key_size | kv_heads * key_size |
+    kv_heads * value_size | gate]``.  ``bias`` (float32) is added to the channels in front of the gate, which then pass
+    ``conv_weight [channels, taps]`` (float32, the current token's tap last; None: no convolution) over the
+    tokens of each request, continued from and into ``conv_state [slots, taps - 1, channels]`` (float32, the
+    biased inputs, oldest first; a view whose slot stride may be larger; not needed with one tap).  Rotation, ``slots``
+    and the caches as in :func:`qkv_norm_store`, of the convolved values.  ``gate_out`` (q_out's dtype,
+    ``[tokens, heads * value_size]``) receives the gate's columns.  ``single_tokens``: every request brings one
+    token, and one launch does it all; otherwise a second one moves the state on."""
+    global launch_count
+    tokens, width = qkv.shape[-2:]
+    channels = (num_heads + num_kv_heads) * key_size + num_kv_heads * value_size
+    gated = num_heads * value_size
+    splits, stride = _maybe_split(qkv, tokens, width, "qkv")
+    if width not in (channels, channels + gated):
+        raise ValueError(f"rows of {width} for {channels} channels and a gate of {gated}")
+    if q_out.numel() != tokens * num_heads * key_size or not q_out.is_contiguous():
+        raise ValueError("q_out must hold [tokens, heads, key_size]")
+    if max(key_size, value_size) > MAX_HEAD_SIZE:
+        raise UnsupportedSize(f"head sizes up to {MAX_HEAD_SIZE}, got {key_size}, {value_size}")
+    if bias is not None and bias.shape != (channels,):
+        raise ValueError(f"bias must be float32 [{channels}]")
+    taps, state_ptr, state_stride, num_slots = 1, 0, 0, 0
+    if conv_weight is not None:
+        taps = conv_weight.shape[1]
+        if conv_weight.shape != (channels, taps):
+            raise ValueError(f"conv weight must be float32 {(channels, taps)}")
+        if not 1 <= taps <= MAX_CONV_TAPS:
+            raise UnsupportedSize(f"the convolution kernels take 1 to {MAX_CONV_TAPS} taps, not {taps}")
+        if taps > 1:
+            if conv_state is None or conv_state.dtype != torch.float32 or conv_state.shape[1:] != (taps - 1, channels) \
+                    or conv_state.stride(2) != 1 or (taps > 2 and conv_state.stride(1) != channels):
+                raise ValueError(f"conv_state must be float32 [slots, {taps - 1}, {channels}] with contiguous slots")
+            if not conv_state.is_cuda:
+                raise KernelError("conv_state must be on a CUDA device: there is no CPU path")
+            state_ptr, state_stride, num_slots = conv_state.data_ptr(), conv_state.stride(0), conv_state.shape[0]
+    page_size = num_pages = 0
+    k_ptr = v_ptr = 0
+    if num_kv_heads and slots is not None:
+        if k_cache is None or v_cache is None:
+            raise ValueError("slots given without caches")
+        num_pages, kvh, page_size, size = k_cache.shape
+        if (kvh, size) != (num_kv_heads, key_size) or v_cache.shape != (num_pages, kvh, page_size, value_size):
+            raise ValueError(
+                f"caches are {tuple(k_cache.shape)} and {tuple(v_cache.shape)}, expected "
+                f"[pages, {num_kv_heads}, page, {key_size}] and [..., {value_size}]"
+            )
+        if k_cache.dtype != q_out.dtype or v_cache.dtype != q_out.dtype:
+            raise TypeError("cache dtype differs from q_out")
+        k_ptr, v_ptr = _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache")
+    pairs = 0
+    if inv_freq is not None and inv_freq.shape[0]:
+        pairs = inv_freq.shape[0]
+        if positions is None or 2 * pairs > key_size:
+            raise ValueError("a rotation needs positions and at most key_size / 2 frequencies")
+    if gate_out is not None and (width == channels or gate_out.shape != (tokens, gated) or gate_out.dtype != q_out.dtype):
+        raise ValueError(f"gate_out must be {q_out.dtype} {(tokens, gated)} and the rows must hold a gate")
+    fn = _fn(
+        "einf_qkv_conv_store",
+        [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int,
+         c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+         c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p],
+    )
+    _check(
+        fn(_dev(qkv, "qkv"), _code(qkv), splits, stride, width, _code(q_out), _opt(bias, "bias", torch.float32),
+           _opt(conv_weight, "conv_weight", torch.float32), taps, state_ptr, state_stride, num_slots,
+           _opt(seq_of_token, "seq_of_token", torch.int32), _opt(q_start, "q_start", torch.int32),
+           _opt(state_slots, "state_slots", torch.int32), state_slots.shape[0],
+           _opt(slots, "slots", torch.int32) if k_ptr else 0, _dev(q_out, "q_out"), k_ptr, v_ptr, tokens, num_heads,
+           num_kv_heads, key_size, value_size, page_size, num_pages,
+           _opt(positions, "positions", torch.int32) if pairs else 0,
+           _opt(inv_freq, "inv_freq", torch.float32) if pairs else 0, pairs, 1 if interleaved else 0,
+           0 if gate_out is None else _dev(gate_out, "gate_out"), 1 if single_tokens else 0, _dev(status, "status"),
+           _stream()),
+        "qkv_conv_store",
+    )
+    if taps > 1 and not single_tokens:
+        launch_count += 1      # the state of the convolutions
+
+
 # ---------------------------------------------------------------------------
 # Latent attention
 def latent_down_store(
@@ -1081,14 +1215,15 @@ ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
 def router_topk(logits: torch.Tensor, top_k: int, score: str, renormalise: bool, expert_ids: torch.Tensor,
                 weights: torch.Tensor, num_experts: Optional[int] = None, correction: Optional[torch.Tensor] = None,
                 groups: Optional[Tuple[int, int]] = None, group_best: int = 1, renormalise_eps: float = 0.0,
-                weight_scale: float = 1.0) -> None:
+                weight_scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
     """Per row of float32 ``logits [tokens, width]`` (or split-K partial sums ``[splits, tokens, width]``,
     added up here): the ``top_k`` experts with the largest scores
     (ties to the lower index) into ``expert_ids`` (int32) and their weights into ``weights`` (float32),
     both ``[tokens, top_k]``, best first.  A weight is ``sigmoid(z)`` or the softmax over all experts;
     ``renormalise`` divides the chosen weights by their sum plus ``renormalise_eps``; ``weight_scale``
     multiplies them at the end.  The experts are the first ``num_experts``
-    columns of a row (default: all of them; further columns belong to someone else).  With
+    columns of a row (default: all of them; further columns belong to someone else).  ``bias`` (float32
+    ``[num_experts]``) is added to their logits.  With
     ``correction`` (float32 ``[num_experts]``) the choice goes by ``score + correction`` while the weights
     stay the scores.  With ``groups = (count, keep)`` the experts form ``count`` equal groups of
     neighbours and only those of the ``keep`` groups whose best choice score is largest can be chosen;
@@ -1104,6 +1239,8 @@ def router_topk(logits: torch.Tensor, top_k: int, score: str, renormalise: bool,
         raise UnsupportedSize(f"top_k {top_k} of {experts} experts (at most 1024) in rows of {width}")
     if correction is not None and (correction.dtype != torch.float32 or correction.shape != (experts,)):
         raise ValueError(f"correction must be float32 [{experts}]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape != (experts,)):
+        raise ValueError(f"bias must be float32 [{experts}]")
     count, keep = (0, 0) if groups is None else (int(groups[0]), int(groups[1]))
     if groups is not None:
         if count <= 0 or experts % count or not 0 < keep <= count or top_k > keep * (experts // count):
@@ -1111,11 +1248,12 @@ def router_topk(logits: torch.Tensor, top_k: int, score: str, renormalise: bool,
     if group_best not in (1, 2):
         raise ValueError(f"a group is scored by its best one or two experts, not {group_best}")
     fn = _fn("einf_router_topk", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                  c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
+                                  c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
     _check(
         fn(_dev(logits, "logits"), splits, stride, tokens, width, experts, top_k, ROUTER_SCORES[score],
            1 if renormalise else 0, float(renormalise_eps), float(weight_scale),
-           _opt(correction, "correction", torch.float32), count, keep, int(group_best),
+           _opt(bias, "bias", torch.float32), _opt(correction, "correction", torch.float32), count, keep,
+           int(group_best),
            _dev(expert_ids, "expert_ids"), _dev(weights, "weights"), _stream()),
         "router_topk",
     )
@@ -1754,6 +1892,63 @@ def norm_conv(
     )
 
 
+def _norm_constants(norm: Optional[tuple], hidden: int, name: str) -> tuple[int, float]:
+    """Pointer of the weight and eps of an RMS norm given as (weight, eps), or (0, 0)."""
+    if norm is None:
+        return 0, 0.0
+    weight, eps = norm
+    if weight.dtype != torch.float32 or weight.shape != (hidden,):
+        raise ValueError(f"the weight of {name} must be float32 [{hidden}]")
+    return _dev(weight, name), float(eps)
+
+
+def stream_norm(pending, pending_scale: float, pending_norm: Optional[tuple], residual: torch.Tensor,
+                norm: Optional[tuple], out: Optional[torch.Tensor]) -> None:
+    """``y = sum(pending)`` (a list of up to two tensors, each ``[T, H]`` or partial sums ``[S, T, H]``; None or
+    empty: nothing is added), ``residual += pending_scale * y``, with ``pending_norm = (weight, eps)`` of its RMS norm
+    ``y * rsqrt(mean(y^2) + eps) * weight`` instead of y; then ``out`` is the RMS norm ``norm = (weight, eps)`` of the
+    residual stream, or the stream itself without ``norm`` (rounded), or nothing (None).  Everything is
+    32-bit; ``out`` is rounded once."""
+    tokens, hidden = residual.shape
+    if residual.dtype != torch.float32:
+        raise TypeError("the residual stream is float32")
+    if hidden > 16384:
+        raise UnsupportedSize(f"stream_norm keeps a row on chip; width {hidden} > 16384")
+    if out is not None and out.shape != (tokens, hidden):
+        raise ValueError(f"out is {tuple(out.shape)}, expected {(tokens, hidden)}")
+    if norm is not None and out is None:
+        raise ValueError("a norm of the stream without an output")
+    fn = _fn(
+        "einf_stream_norm",
+        [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_longlong, c_float, c_void_p, c_float, c_void_p,
+         c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+    )
+    _check(
+        fn(*_pending_terms(pending, tokens, hidden), float(pending_scale),
+           *_norm_constants(pending_norm, hidden, "pending_norm"), _dev(residual, "residual"),
+           *_norm_constants(norm, hidden, "norm"), 0 if out is None else _dev(out, "out"),
+           FLOAT32 if out is None else _code(out), tokens, hidden, _stream()),
+        "stream_norm",
+    )
+
+
+def side_gate(product: torch.Tensor, table: torch.Tensor, token_ids: torch.Tensor, out: torch.Tensor) -> None:
+    """``out[t] = gelu(product[t]) * table[token_ids[t]]`` with the tanh form of GELU: ``product [T, n]`` or float32
+    partial sums ``[S, T, n]`` of it, ``table [vocab, n]``."""
+    tokens, size = out.shape
+    splits, stride = _maybe_split(product, tokens, size, "product")
+    if table.shape[1] != size:
+        raise ValueError(f"table is {tuple(table.shape)}, expected [vocab, {size}]")
+    fn = _fn("einf_side_gate", [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                                c_int, c_void_p])
+    _check(
+        fn(_dev(product, "product"), _code(product), splits, stride, _dev(table, "table"), _code(table),
+           _opt(token_ids, "token_ids", torch.int32), _dev(out, "out"), _code(out), tokens, size, table.shape[0],
+           _stream()),
+        "side_gate",
+    )
+
+
 def stream_tail(
     residual: torch.Tensor,
     pending,
@@ -1761,9 +1956,11 @@ def stream_tail(
     token_ids: torch.Tensor,
     side: Optional[tuple],
     depth: Optional[tuple],
+    pending_norm: Optional[tuple] = None,
 ) -> None:
     """The end of a layer in one pass over every row of the stream, in 32-bit:
-    ``x = residual + pending_scale * sum(pending)`` (as in :func:`norm_conv`); with ``side = (table
+    ``x = residual + pending_scale * sum(pending)`` (as in :func:`norm_conv`; with ``pending_norm`` through a norm, as
+    in :func:`stream_norm`); with ``side = (table
     [vocab, n], gate [n, H], proj_t [n, H], norm [H] float32, eps)``: ``g = gelu(gate x) * table[token]``,
     ``y = proj_t^T g``, ``x += pending_scale * y * rsqrt(mean(y^2) + eps) * norm``; with ``depth =
     (history [L + 1, T, H] float32, index, weight [index + 2] float32)``: ``history[index + 1] = x`` and
@@ -1795,11 +1992,12 @@ def stream_tail(
         "einf_stream_tail",
         [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_longlong, c_float, c_void_p,
          c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_longlong,
-         c_int, c_int, c_void_p],
+         c_void_p, c_float, c_int, c_int, c_void_p],
     )
     _check(
         fn(_dev(residual, "residual"), *_pending_terms(pending, tokens, hidden), float(pending_scale),
-           _opt(token_ids, "token_ids", torch.int32), *side_args, *depth_args, tokens, hidden, _stream()),
+           _opt(token_ids, "token_ids", torch.int32), *side_args, *depth_args,
+           *_norm_constants(pending_norm, hidden, "pending_norm"), tokens, hidden, _stream()),
         "stream_tail",
     )
 
@@ -2372,6 +2570,7 @@ def paged_decode_attention_auto(
     keep_first: int = 0,
     sink: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None,
+    value_gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Decode attention by the kernel, cluster size and number of clusters per token that
     ``decode_plan`` picks for this batch; ``max_context`` is the longest context among the
@@ -2385,8 +2584,8 @@ def paged_decode_attention_auto(
     if kernel == "tcgen05":
         paged_decode_attention_tcgen05(q, k_cache, v_cache, block_table, seq_of_token, positions, out, scale, window,
                                        cluster, status, token_list, splits, chunk=chunk, softcap=softcap,
-                                       keep_first=keep_first, sink=sink, gate=gate)
-    elif chunk or softcap or (window and keep_first) or sink is not None or gate is not None:
+                                       keep_first=keep_first, sink=sink, gate=gate, value_gate=value_gate)
+    elif chunk or softcap or (window and keep_first) or sink is not None or gate is not None or value_gate is not None:
         raise UnsupportedSize("a chunked mask, a soft cap, kept first positions, a sink or a gate need the tcgen05 "
                               "decode kernel (head size 64 or 128)")
     else:
@@ -2477,6 +2676,7 @@ def paged_decode_attention_tcgen05(
     keep_first: int = 0,
     sink: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None,
+    value_gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Decode attention on the tcgen05 tensor cores with the keys as the 128-row operand
     (S^T = K Q^T, O^T = V^T P^T), so the tile is full at any number of query heads.  Key splits
@@ -2506,7 +2706,7 @@ def paged_decode_attention_tcgen05(
     fn = _fn(
         "einf_paged_decode_attention_tcgen05",
         [c_void_p] * 8 + [c_int] * 6 + [c_float, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
-         c_void_p, c_void_p, c_void_p],
+         c_void_p, c_longlong, c_void_p, c_void_p, c_void_p],
         f"HEAD_SIZE={head_size}",
     )
     _check(
@@ -2518,7 +2718,8 @@ def paged_decode_attention_tcgen05(
            int(keep_first) if window else 0,
            int(chunk) if chunk else 0, float(softcap) if softcap else 0.0, cluster,
            splits, shares.data_ptr() if splits > 1 else None, counters.data_ptr() if splits > 1 else None,
-           _opt(sink, "sink", torch.float32), _opt(gate, "gate", torch.float32), _dev(status, "status"), _stream()),
+           _opt(sink, "sink", torch.float32), _opt(gate, "gate", torch.float32),
+           *_value_gate(value_gate, q, head_size, False), _dev(status, "status"), _stream()),
         "paged_decode_attention_tcgen05",
     )
 
@@ -2582,6 +2783,7 @@ def paged_prefill_attention(
     keep_first: int = 0,
     sink: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None,
+    value_gate: Optional[torch.Tensor] = None,
 ) -> None:
     """Tensor-core causal attention for prompt portions.  ``q_tiles`` is int32 ``[tiles, 4]``:
     request, first token (packed index), rows (at most ``Q_TILE``), position of the first row.
@@ -2591,8 +2793,8 @@ def paged_prefill_attention(
     ``mma.sync`` kernel.  ``prefill_cluster`` (1 to 8; 0: ``prefill_cluster_size`` of the number of
     row tiles and ``cached_before``, the most tokens that a portion of this step finds in the
     cache, if the caller knows it) is the number of CTAs that share a row tile's keys in the
-    tcgen05 kernel.  ``chunk``, ``softcap``, ``sink`` and ``gate`` (see :func:`paged_attention_generic`) are the tcgen05
-    kernel's alone."""
+    tcgen05 kernel.  ``chunk``, ``softcap``, ``sink``, ``gate`` and ``value_gate`` (see :func:`paged_attention_generic`)
+    are the tcgen05 kernel's alone."""
     tokens, num_heads, head_size, num_pages, num_kv_heads, page_size = _check_fast_attention(q, k_cache, v_cache, out)
     if sink is not None and (sink.dtype != torch.float32 or sink.shape != (num_heads,)):
         raise ValueError(f"sink must be float32 [{num_heads}]")
@@ -2611,7 +2813,7 @@ def paged_prefill_attention(
         fn = _fn(
             "einf_paged_prefill_attention_tcgen05",
             [c_void_p] * 5 + [c_int, c_void_p] + [c_int] * 6 + [c_float, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                                                                 c_void_p, c_void_p, c_void_p],
+                                                                 c_void_p, c_void_p, c_longlong, c_void_p, c_void_p],
             f"HEAD_SIZE={head_size}",
         )
         cluster = prefill_cluster
@@ -2629,11 +2831,12 @@ def paged_prefill_attention(
                float(scale), int(window) if window else 0, int(keep_first) if window else 0,
                int(chunk) if chunk else 0,
                float(softcap) if softcap else 0.0, int(cluster), _opt(sink, "sink", torch.float32),
-               _opt(gate, "gate", torch.float32), _dev(status, "status"), _stream()),
+               _opt(gate, "gate", torch.float32), *_value_gate(value_gate, q, head_size, True),
+               _dev(status, "status"), _stream()),
             "paged_prefill_attention_tcgen05",
         )
         return
-    if chunk or softcap or (window and keep_first) or sink is not None or gate is not None:
+    if chunk or softcap or (window and keep_first) or sink is not None or gate is not None or value_gate is not None:
         raise UnsupportedSize("a chunked mask, a soft cap, kept first positions, a sink or a gate need the tcgen05 "
                               "prefill kernel (head size 64 or 128)")
     fn = _fn(

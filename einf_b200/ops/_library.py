@@ -51,6 +51,9 @@ LAUNCHERS = {
     "einf_act_mul": "pointwise",
     "einf_norm_conv": "stream",
     "einf_stream_tail": "stream",
+    "einf_stream_norm": "stream",
+    "einf_side_gate": "stream",
+    "einf_qkv_conv_store": "qkv_conv",
     "einf_hyper_norm": "hyper",
     "einf_paged_attention_mixed": "attention_mixed",
     "einf_paged_attention_mixed_tiled": "attention_mixed_tiled",

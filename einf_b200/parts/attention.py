@@ -29,6 +29,14 @@ weights before any rotation: ``"head"``, one weight of the head's size for all q
 for all key heads; ``"row"``, weights over all heads, and the root mean square is taken over the
 whole projection at once instead of head by head.  ``values: "keys"``: the layer has no value
 projection; a token's values are its keys as projected, before norm and rotation.
+
+``conv_taps`` n: every channel of the projected (and biased) queries, keys and values passes a causal
+convolution over time of n taps, before rotation and cache write; the last n - 1 projected rows of a
+request are state beside the pages (also where the pages are another layer's).  ``sink_score`` s: every
+head's softmax has ``exp(s)`` in its denominator, a constant in the place of a stored ``sink``.
+``output_gate``: the mixed heads are multiplied element by element by ``sigmoid(W_g h)`` before the output
+projection; W_g rides along in the product for queries, keys and values, and the attention kernels
+multiply as they divide by the softmax's sum.
 """
 from __future__ import annotations
 
@@ -36,7 +44,7 @@ import torch
 
 from .. import ops
 from ..config.specs import TensorSpec
-from .base import CacheView, Mixer, PagedKVNeed, StepContext, build_nested, register_part
+from .base import CacheView, Mixer, PagedKVNeed, PagesAndState, StateNeed, StepContext, build_nested, register_part
 
 
 @register_part("mixer", "attention")
@@ -66,6 +74,14 @@ class PagedAttention(Mixer):
                 specs["v_proj.bias"] = TensorSpec((kv_heads * value_size,), "bias")
         if spec.get("out_bias", False):
             specs["o_proj.bias"] = TensorSpec((hidden,), "bias")
+        if spec.get("conv_taps"):
+            channels = {"q_conv.weight": heads * size}
+            if own_kv:
+                channels.update({"k_conv.weight": kv_heads * size, "v_conv.weight": kv_heads * value_size})
+            for name, count in channels.items():
+                specs[name] = TensorSpec((count, spec["conv_taps"]), "conv")
+        if spec.get("output_gate"):
+            specs["gate_proj.weight"] = TensorSpec((heads * value_size, hidden))
         if spec.get("value_mix"):
             specs["value_mix"] = TensorSpec((), "fraction")   # stored by the source layer too, unused there
         if spec.get("talking_heads"):
@@ -90,6 +106,7 @@ class PagedAttention(Mixer):
             or spec["position"].get("layout", "halves") != "halves"
             or PagedAttention._mixes_scores(spec) or spec.get("output_scale") is not None
             or spec.get("sink") or spec.get("values", "projected") != "projected"
+            or spec.get("conv_taps") or spec.get("sink_score") is not None or spec.get("output_gate")
         )
 
     @staticmethod
@@ -109,7 +126,8 @@ class PagedAttention(Mixer):
         if cls._is_general(spec):
             fast = (f"attention_tcgen05:HEAD_SIZE={int(spec['head_size'])}",) \
                 if cls._general_on_tensor_cores(spec, runtime.dtype) else ()
-            return ("pointwise", "attention_generic", "gemm_simt") + cls._product_libraries(runtime) + fast
+            store = ("qkv_conv",) if spec.get("conv_taps") or spec.get("output_gate") else ("pointwise",)
+            return store + ("attention_generic", "gemm_simt") + cls._product_libraries(runtime) + fast
         if ops.has_fast_attention(runtime.dtype, int(spec["head_size"])):
             # the page size is the engine's choice: ask for both prefill kernels of this head size
             libraries = ops.attention_libraries(int(spec["head_size"]), 16)
@@ -176,7 +194,8 @@ class PagedAttention(Mixer):
             names = ["q_proj", "k_proj"]
         else:
             names = ["q_proj", "k_proj", "v_proj"]
-        matrices = [tensors[n + ".weight"] for n in names]
+        self.output_gate = bool(spec.get("output_gate"))
+        matrices = [tensors[n + ".weight"] for n in names + (["gate_proj"] if self.output_gate else [])]
         if len({m.dtype for m in matrices}) > 1:
             matrices = [m.to(torch.float32) for m in matrices]
         self.qkv_weight = runtime.matrix(torch.cat(matrices, dim=0))
@@ -214,23 +233,48 @@ class PagedAttention(Mixer):
                 raise ValueError("a layer that mixes its heads' scores has no weighted norm and values of its own")
         elif self.output_scale != 1.0:
             raise ValueError("output_scale is applied by the score-mixing kernel only")
-        if spec.get("sink"):
+        if spec.get("sink") or spec.get("sink_score") is not None:
             if self.softcap or self.chunk or self.keep_first:
                 raise ValueError("a sink comes without a soft cap, chunks or kept positions")
-            self.sink = runtime.vector(tensors["sink"])
+            if spec.get("sink_score") is None:
+                self.sink = runtime.vector(tensors["sink"])
+            elif spec.get("sink") or self.mixes_scores:
+                raise ValueError("a constant sink comes without a stored one and without mixed scores")
+            else:
+                self.sink = torch.full((self.num_heads,), float(spec["sink_score"]), dtype=torch.float32,
+                                       device=runtime.device)
+        self.conv_taps = int(spec.get("conv_taps") or 0)
+        self.conv_weight = None
+        if self.conv_taps or self.output_gate:
+            if self.qk_unit_eps is not None or self.value_mix or self.values_from_keys or self.mixes_scores:
+                raise ValueError("convolved projections or an output gate come without normed heads, mixed values or scores")
+        if self.conv_taps:
+            if self.conv_taps > ops.MAX_CONV_TAPS:
+                raise ops.UnsupportedSize(f"{self.conv_taps} taps: the convolution kernels take 1 to {ops.MAX_CONV_TAPS}")
+            self.conv_weight = runtime.vector(torch.cat(
+                [tensors[n.replace("_proj", "_conv") + ".weight"].float() for n in names], dim=0))
+        #: channels of the projected queries, and keys and values where the layer has its own
+        self.channels = sum(tensors[n + ".weight"].shape[0] for n in names)
         self.fast = not self.general and ops.has_fast_attention(runtime.dtype, self.head_size)
         self.general_fast = self.general and not self.mixes_scores and self._general_on_tensor_cores(spec, runtime.dtype)
 
     def cache_need(self):
         value = self.value_size if self.value_size != self.head_size else None
-        return PagedKVNeed(self.num_kv_heads, self.head_size, self.window, value, self.keep_first)
+        pages = PagedKVNeed(self.num_kv_heads, self.head_size, self.window, value, self.keep_first)
+        if self.conv_taps < 2:
+            return pages
+        # the convolutions' last taps - 1 inputs, oldest first
+        return PagesAndState(pages, StateNeed(((self.conv_taps - 1) * self.channels,), torch.float32))
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
         tokens = x.shape[0]
         dtype, device = self.runtime.dtype, x.device
         qkv = ops.project(x, self.qkv_weight, ctx.status)   # [T, width], or split-K partial sums
         q = torch.empty((tokens, self.num_heads, self.head_size), dtype=dtype, device=device)
-        if self.general:
+        gate = None
+        if self.conv_taps or self.output_gate:
+            gate = self._convolve_and_store(qkv, q, ctx, cache)
+        elif self.general:
             writes = cache.writes and cache.k is not None and not self.shared_kv
             shared_values = None
             if self.value_mix == "source":
@@ -256,12 +300,35 @@ class PagedAttention(Mixer):
                 qkv, self.qkv_bias, ctx, cache, q, self.num_heads, self.num_kv_heads, self.head_size
             )
         mixed = torch.empty((tokens, self.num_heads, self.value_size), dtype=dtype, device=device)
-        self.attend(q, ctx, cache, mixed)
+        self.attend(q, ctx, cache, mixed, gate)
         if self.out_bias is None:
             return ops.project(mixed.view(tokens, -1), self.out_weight, ctx.status)
         out = torch.empty((tokens, self.hidden_size), dtype=dtype, device=device)
         ops.linear(mixed.view(tokens, -1), self.out_weight, self.out_bias, out)
         return out
+
+    def _convolve_and_store(self, qkv, q, ctx: StepContext, cache: CacheView):
+        """Queries into ``q``, keys and values into the pages; returns the logits of the output gate
+        ``[T, heads * value_size]`` (None without one)."""
+        tokens, gated = q.shape[0], self.num_heads * self.value_size
+        writes = cache.writes and cache.k is not None and not self.shared_kv
+        gate = copy = None
+        if self.output_gate:
+            if ops.gate_in_place(qkv, self.channels, self.runtime.dtype):
+                gate = qkv[:, self.channels:]                 # left where the product put it
+            else:
+                gate = copy = torch.empty((tokens, gated), dtype=self.runtime.dtype, device=q.device)
+        state = None
+        if self.conv_taps > 1:
+            state = cache.state[:, :(self.conv_taps - 1) * self.channels].unflatten(1, (self.conv_taps - 1, self.channels))
+        ops.qkv_conv_store(
+            qkv, self.qkv_bias, self.conv_weight, state, ctx.seq_of_token, ctx.q_start, ctx.state_slots,
+            ctx.slots[cache.group] if writes else None, q, cache.k if writes else None, cache.v if writes else None,
+            self.num_heads, 0 if self.shared_kv else self.num_kv_heads, self.head_size, self.value_size, ctx.status,
+            positions=ctx.positions, inv_freq=self.position.inv_freq,
+            interleaved=getattr(self.position, "interleaved", False), gate_out=copy, single_tokens=ctx.decode_only,
+        )
+        return gate
 
     def launch_key(self, ctx: StepContext, page_size: int) -> tuple:
         """The decode attention cuts a token's keys by the number of single tokens and the bucket
@@ -282,7 +349,7 @@ class PagedAttention(Mixer):
         return ("attention", self.num_heads, self.num_kv_heads, self.head_size, self.window, self.fast, self.general,
                 self.mixes_scores)
 
-    def attend(self, q, ctx: StepContext, cache: CacheView, out) -> None:
+    def attend(self, q, ctx: StepContext, cache: CacheView, out, gate=None) -> None:
         """bfloat16 with a head size up to 128 (a layer with a chunked mask, a soft cap or unit-norm
         heads: head sizes 64 and 128 with values as large as keys): the tensor-core kernels, cluster decode for the
         requests that bring one token, tiled prefill for the others, side by side in a mixed batch.  Everything else (the 32-bit path,
@@ -303,17 +370,17 @@ class PagedAttention(Mixer):
                     q, cache.k, cache.v, table, ctx.seq_of_token, ctx.positions, out, self.scale,
                     self.window, ctx.status, None if ctx.decode_only else ctx.single_tokens,
                     max_context=ctx.max_context_len, chunk=self.chunk, softcap=self.softcap,
-                    keep_first=self.keep_first, sink=self.sink,
+                    keep_first=self.keep_first, sink=self.sink, value_gate=gate,
                 )
             if ctx.q_tiles.shape[0]:
                 ops.paged_prefill_attention(
                     q, cache.k, cache.v, table, ctx.q_tiles, out, self.scale, self.window, ctx.status,
                     cached_before=ctx.max_portion_start, chunk=self.chunk, softcap=self.softcap,
-                    keep_first=self.keep_first, sink=self.sink,
+                    keep_first=self.keep_first, sink=self.sink, value_gate=gate,
                 )
             return
         ops.paged_attention_generic(
             q, cache.k, cache.v, ctx.block_tables[cache.group], ctx.seq_of_token, ctx.positions,
             out, self.scale, self.window, ctx.status, chunk=self.chunk, softcap=self.softcap,
-            keep_first=self.keep_first, sink=self.sink,
+            keep_first=self.keep_first, sink=self.sink, value_gate=gate,
         )

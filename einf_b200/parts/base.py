@@ -168,7 +168,8 @@ class CacheView:
 
     ``k`` and ``v`` are ``[pages, kv_heads, page_size, head_size]`` for a paged
     need; ``state`` is ``[slots, *shape]`` for a state need.  ``writes`` is false
-    for a run that reads another run's cache.
+    for a run that reads another run's cache (of a run with pages and state, another run's
+    pages: the state row is its own all the same).
     """
 
     group: int = -1

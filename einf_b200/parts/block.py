@@ -103,7 +103,8 @@ def build_block(layer_spec, tensors, runtime) -> Block:
 @register_part("block", "prenorm_stream")
 class PreNormStreamBlock(Block):
     """``h += m mixer(c1(norm1(h))); h += m ff(c2(norm2(h)))`` with a residual multiplier m and, each
-    optional: a short causal convolution ``c(x) = x + conv(x)`` in front of a sublayer (run in the
+    optional: a norm behind a sublayer (``m norm(mixer(..))``; run in the launch that adds the sublayer's output
+    to the stream), a short causal convolution ``c(x) = x + conv(x)`` in front of a sublayer (run in the
     launch of the norm before it, continued from and into the request's state row), no feed-forward,
     a per-layer token input added after the feed-forward, and a weighted sum over the results of
     all layers so far in place of the layer's own result.  The layer's last kernel adds the pending
@@ -111,8 +112,12 @@ class PreNormStreamBlock(Block):
     hands nothing pending to the next one.  The block's state row holds the convolutions' inputs
     in front of whatever state its mixer keeps."""
 
-    optional_roles = ("mixer_conv", "feed_forward_norm", "feed_forward_conv", "feed_forward", "token_input",
-                      "depth_mix")
+    optional_roles = ("mixer_conv", "mixer_post_norm", "feed_forward_norm", "feed_forward_conv", "feed_forward",
+                      "feed_forward_post_norm", "token_input", "depth_mix")
+
+    #: from this many tokens on the token input's two matrices are products of their own instead of
+    #: part of the layer's last kernel
+    SIDE_PRODUCT_TOKENS = 128
 
     @classmethod
     def part_categories(cls):
@@ -120,9 +125,11 @@ class PreNormStreamBlock(Block):
             "mixer_norm": "norm",
             "mixer_conv": "stream",
             "mixer": "mixer",
+            "mixer_post_norm": "norm",
             "feed_forward_norm": "norm",
             "feed_forward_conv": "stream",
             "feed_forward": "feed_forward",
+            "feed_forward_post_norm": "norm",
             "token_input": "stream",
             "depth_mix": "stream",
         }
@@ -142,6 +149,11 @@ class PreNormStreamBlock(Block):
             raise ValueError("a feed-forward and its norm come together")
         if self.feed_forward is None and self.feed_forward_conv is not None:
             raise ValueError("a convolution in front of a feed-forward that is not there")
+        if self.feed_forward is None and self.feed_forward_post_norm is not None:
+            raise ValueError("a norm behind a feed-forward that is not there")
+        for norm in (self.mixer_norm, self.mixer_post_norm, self.feed_forward_norm, self.feed_forward_post_norm):
+            if norm is not None and (norm.centre or norm.bias is not None):
+                raise ValueError("a prenorm_stream layer has RMS norms without bias")
         needs = [conv.state_need() if conv is not None else None for conv in (self.mixer_conv, self.feed_forward_conv)]
         self._need, offsets = join_needs(*needs, self.mixer.cache_need())
         self._conv_offsets, self._mixer_offset = offsets[:2], offsets[2]
@@ -157,16 +169,40 @@ class PreNormStreamBlock(Block):
         rows = cache.state[:, offset:offset + (conv.taps - 1) * conv.size]
         return rows.unflatten(1, (conv.taps - 1, conv.size))
 
-    def _normalise(self, which: int, pending, residual, ctx, cache):
+    def _normalise(self, which: int, pending, post, residual, ctx, cache):
+        """Add what is pending (through the norm ``post`` behind its sublayer, if there is one) and return what
+        the next sublayer reads."""
         norm = (self.mixer_norm, self.feed_forward_norm)[which]
         conv = (self.mixer_conv, self.feed_forward_conv)[which]
         out = torch.empty(residual.shape, dtype=self.runtime.dtype, device=residual.device)
+        if conv is None:
+            ops.stream_norm(pending, self.residual_mult, self._constants(post), residual, self._constants(norm), out)
+            return out
+        if pending is not None and post is not None:
+            ops.stream_norm(pending, self.residual_mult, self._constants(post), residual, None, None)
+            pending = None
         ops.norm_conv(
-            pending, self.residual_mult, residual, norm.weight, norm.eps, None if conv is None else conv.weight,
+            pending, self.residual_mult, residual, norm.weight, norm.eps, conv.weight,
             self._conv_state(which, cache), ctx.seq_of_token, ctx.q_start, ctx.state_slots, out,
             single_tokens=ctx.decode_only,
         )
         return out
+
+    @staticmethod
+    def _constants(norm):
+        return None if norm is None else (norm.weight, norm.eps)
+
+    def _add_token_input(self, terms, post, residual, ctx):
+        """The end of a layer at prompt sizes: the token input's two matrices on the tensor cores, between a
+        kernel that adds the pending output and one that adds the token input."""
+        side, tokens = self.token_input, residual.shape[0]
+        x = torch.empty(residual.shape, dtype=self.runtime.dtype, device=residual.device)
+        ops.stream_norm(terms, self.residual_mult, self._constants(post), residual, None, x)
+        product = ops.project(x, side.gate, ctx.status)
+        g = torch.empty((tokens, side.size), dtype=self.runtime.dtype, device=residual.device)
+        ops.side_gate(product, side.table, ctx.token_ids, g)
+        y = ops.project(g, side.proj_rows, ctx.status)
+        ops.stream_norm([y], self.residual_mult, (side.norm, side.eps), residual, None, None)
 
     def forward(self, residual, pending, ctx, cache):
         if pending is not None:
@@ -177,21 +213,25 @@ class PreNormStreamBlock(Block):
             history = depth.history(ctx, residual)
             if depth.index == 0:
                 history[0].copy_(residual)      # the embedding output, before this layer changes the stream
-        x = self._normalise(0, None, residual, ctx, cache)
+        x = self._normalise(0, None, None, residual, ctx, cache)
         view = cache
         if self._mixer_offset is not None:
             view = CacheView(cache.group, cache.k, cache.v, cache.state[:, self._mixer_offset:], cache.writes,
                              cache.page_size)
         terms = self.mixer.forward_terms(x, ctx, view) if hasattr(self.mixer, "forward_terms") \
             else [self.mixer.forward(x, ctx, view)]
+        post = self.mixer_post_norm
         if self.feed_forward is not None:
-            x = self._normalise(1, terms, residual, ctx, cache)
-            terms = [self.feed_forward.forward(x, ctx)]
+            x = self._normalise(1, terms, post, residual, ctx, cache)
+            terms, post = [self.feed_forward.forward(x, ctx)], self.feed_forward_post_norm
         side = self.token_input
+        if side is not None and depth is None and residual.shape[0] >= self.SIDE_PRODUCT_TOKENS:
+            self._add_token_input(terms, post, residual, ctx)
+            return None
         ops.stream_tail(
             residual, terms, self.residual_mult, ctx.token_ids,
             None if side is None else (side.table, side.gate, side.proj, side.norm, side.eps),
-            None if depth is None else (history, depth.index, depth.weight),
+            None if depth is None else (history, depth.index, depth.weight), pending_norm=self._constants(post),
         )
         return None
 

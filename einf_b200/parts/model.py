@@ -54,11 +54,13 @@ def kernel_libraries(model_spec: ModelSpec, runtime: Runtime) -> tuple[str, ...]
 
 @dataclass(frozen=True)
 class EntryCache:
-    """Cache of one schedule entry: ``owner`` is the entry whose storage it uses."""
+    """Cache of one schedule entry: ``owner`` is the entry whose storage it uses.  The state row of an
+    entry that needs pages and state is its own, also where it reads another entry's pages."""
 
     need: PagedKVNeed | StateNeed | PagesAndState | None
     owner: int
     group: int = -1   # page group of a paged need
+    state_owner: int = -1   # the entry whose state row it uses (-1: it has none)
 
 
 @dataclass(frozen=True)
@@ -97,38 +99,46 @@ class DecoderModel:
     def _plan_cache(self) -> CachePlan:
         windows: list[tuple[Optional[int], int]] = []
         entries: list[EntryCache] = []
-        for index, entry in enumerate(self.schedule):
-            block = self.blocks[entry.layer]
-            # a block that keeps something of its own beside its mixer's cache says so itself
-            need = block.cache_need() if hasattr(block, "cache_need") else block.mixer.cache_need()
-            owner = index if entry.cache_from is None else entry.cache_from
+        blocks = [self.blocks[entry.layer] for entry in self.schedule]
+        # a block that keeps something of its own beside its mixer's cache says so itself
+        needs = [b.cache_need() if hasattr(b, "cache_need") else b.mixer.cache_need() for b in blocks]
+        owners = [index if entry.cache_from is None else entry.cache_from for index, entry in enumerate(self.schedule)]
+        for index, (need, owner) in enumerate(zip(needs, owners)):
+            paged, state = pages_of(need), state_of(need)
             if owner != index:
-                owner_need = entries[owner].need
-                if isinstance(need, PagesAndState):
-                    raise ValueError(f"schedule entry {index} carries a state row and cannot read another entry's cache")
-                if type(owner_need) is not type(need) or (
-                    isinstance(need, PagedKVNeed)
-                    and (need.num_kv_heads, need.head_size, need.value_size)
-                    != (owner_need.num_kv_heads, owner_need.head_size, owner_need.value_size)
-                ):
+                theirs = pages_of(needs[owner])
+                if paged is None or theirs is None:
+                    fits = type(needs[owner]) is type(need)
+                else:
+                    fits = (paged.num_kv_heads, paged.head_size, paged.value_size) == \
+                        (theirs.num_kv_heads, theirs.head_size, theirs.value_size)
+                if not fits:
                     raise ValueError(
-                        f"schedule entry {index} cannot read the cache of entry {owner}: {need} vs {owner_need}"
+                        f"schedule entry {index} cannot read the cache of entry {owner}: {need} vs {needs[owner]}"
                     )
             group = -1
-            paged = pages_of(need)
             if paged is not None:
                 if owner != index:
                     group = entries[owner].group
                 else:
-                    # a group is a window and the first positions it keeps
-                    key = (paged.window, paged.keep_first if paged.window else 0)
+                    # a group is a window and the first positions it keeps: as far back as any entry
+                    # that reads these pages sees
+                    key = self._kept_range([pages_of(n) for n, o in zip(needs, owners) if o == index])
                     if key not in windows:
                         windows.append(key)
                     group = windows.index(key)
-            entries.append(EntryCache(need, owner, group))
+            state_owner = -1 if state is None else (owner if paged is None else index)
+            entries.append(EntryCache(need, owner, group, state_owner))
         if not windows:
             windows.append((None, 0))  # the manager always has one page group
         return CachePlan(tuple(entries), tuple(w for w, _ in windows), tuple(k for _, k in windows))
+
+    @staticmethod
+    def _kept_range(readers) -> tuple[Optional[int], int]:
+        """Window and kept first positions of the pages that all these needs are served from."""
+        if any(not need.window for need in readers):
+            return None, 0
+        return max(need.window for need in readers), max(need.keep_first for need in readers)
 
     def forward(self, ctx: StepContext, caches: list[CacheView]) -> torch.Tensor:
         """Run the step's tokens through every schedule entry; float logits ``[S, vocab]``

@@ -3,11 +3,13 @@
 ``routed_mlp``: router logits ``z = W_router x`` in 32-bit; the ``top_k`` experts with the largest
 scores (``score``: ``sigmoid`` or ``softmax`` over all experts; ``renormalise`` divides the chosen
 weights by their sum, to which ``renormalise_eps`` is added; ``weight_scale`` multiplies the weights);
-an expert is ``down(silu(gate(u)) * up(u))`` without biases.  With
+an expert is ``down(silu(gate(u)) * up(u))`` without biases, or with what ``activation`` names in the place
+of SiLU (see :class:`~einf_b200.parts.mlp.GateActivation`; ``shared_activation`` for the shared expert).  With
 ``weight_on: "input"`` the expert sees ``u = w x`` and its output is added as it is; with ``"output"``
 it sees x and its output is multiplied by w.
 
-Optional, each from the spec.  ``correction``: a stored number per router output that is added to the
+Optional, each from the spec.  ``router_bias``: a stored number per router output that is added to its
+logit.  ``correction``: a stored number per router output that is added to the
 scores for the choice alone (the weights stay the scores).  ``groups`` (``count``, ``keep``): the router's
 outputs form equal groups of neighbours, and only those of the ``keep`` groups whose best choice score
 is largest can be chosen (with ``best`` 2 in the groups: whose two best together are largest).  ``num_identity``: the router has that many outputs beyond the experts;
@@ -29,6 +31,7 @@ import torch
 from .. import ops
 from ..config.specs import TensorSpec
 from .base import FeedForward, register_part
+from .mlp import GateActivation
 
 
 @register_part("feed_forward", "routed_mlp")
@@ -41,6 +44,8 @@ class RoutedMLP(FeedForward):
         hidden, inter, experts = spec["hidden_size"], spec["intermediate_size"], spec["num_experts"]
         outputs = experts + int(spec.get("num_identity") or 0)
         specs = {"router.weight": TensorSpec((outputs, hidden))}
+        if spec.get("router_bias"):
+            specs["router.bias"] = TensorSpec((outputs,), "bias")
         if spec.get("correction"):
             specs["router.correction"] = TensorSpec((outputs,), "small")
         if spec.get("shared"):
@@ -94,6 +99,9 @@ class RoutedMLP(FeedForward):
                 raise ValueError(f"{self.num_outputs} router outputs in {count} groups of which {keep} are kept "
                                  f"cannot give {self.top_k} choices")
         self.correction = runtime.vector(tensors["router.correction"]) if spec.get("correction") else None
+        self.router_bias = runtime.vector(tensors["router.bias"]) if spec.get("router_bias") else None
+        self.activation = GateActivation(spec.get("activation") or "silu")
+        self.shared_activation = GateActivation(spec.get("shared_activation") or "silu")
         self.shared_size = int(spec.get("shared") or 0)
         self.shared_gated = bool(self.shared_size and spec.get("shared_gate"))
         router_rows = [tensors["router.weight"]]
@@ -123,14 +131,14 @@ class RoutedMLP(FeedForward):
         weights = torch.empty((tokens, top_k), dtype=torch.float32, device=device)
         ops.router_topk(logits, top_k, self.score, self.renormalise, expert_ids, weights, self.num_outputs,
                         self.correction, self.groups, group_best=self.group_best,
-                        renormalise_eps=self.renormalise_eps, weight_scale=self.weight_scale)
+                        renormalise_eps=self.renormalise_eps, weight_scale=self.weight_scale, bias=self.router_bias)
         addend_gate = None
         if self.shared_size:
             if add is not None:
                 raise ValueError("a routed feed-forward with a shared expert takes no other addend")
             gate_up = ops.project(x, self.shared_gate_up, ctx.status)
             inner = torch.empty((tokens, self.shared_size), dtype=dtype, device=device)
-            ops.silu_mul(gate_up, inner)
+            self.shared_activation(gate_up, inner)
             add = ops.project(inner, self.shared_down, ctx.status)      # [T, hidden], or partial sums
             if self.shared_gated:
                 addend_gate = (logits, self.num_outputs)
@@ -142,7 +150,7 @@ class RoutedMLP(FeedForward):
         gate_up = torch.empty((rows, 2 * self.intermediate_size), dtype=dtype, device=device)
         ops.moe_gemm(sorted_x, self.gate_up_weight, offsets, gate_up, ctx.status)
         hidden = torch.empty((rows, self.intermediate_size), dtype=dtype, device=device)
-        ops.silu_mul(gate_up, hidden)
+        self.activation(gate_up, hidden)
         splits = 1
         if ops.moe_gemm_on_tensor_cores(hidden, self.down_weight):
             splits = ops.moe_gemm_splits(rows, experts, self.hidden_size, self.intermediate_size)

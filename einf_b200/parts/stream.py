@@ -14,7 +14,8 @@ layer i is ``sum_(j <= i + 1) w[j] X_j``.  The results of all layers of the step
 32-bit buffer in ``ctx.extras``.
 
 The parts hold tensors and sizes; the block that arranges them (``prenorm_stream``) launches one
-kernel for the end of a layer: pending sublayer output, token input and weighted sum together.
+kernel for the end of a layer: pending sublayer output, token input and weighted sum together (at prompt
+sizes without a weighted sum: two products with a kernel in front, between and behind).
 
 ``hyper_connection``: the model has several residual streams x_1 .. x_s instead of one
 (:class:`ResidualStreams`), all equal to the embedding output at the start.  A sublayer reads ``u = sum_s
@@ -67,7 +68,7 @@ class TokenSideInput(Part):
 
     @classmethod
     def kernel_libraries(cls, spec, runtime):
-        return ("stream",)
+        return ("stream", "gemm_simt") + (("gemm_tcgen05",) if runtime.dtype == torch.bfloat16 else ())
 
     def __init__(self, spec, tensors, runtime):
         super().__init__(spec, tensors, runtime)
@@ -79,7 +80,8 @@ class TokenSideInput(Part):
         # this layer's columns of the table only: the layers together hold the table once
         self.table = runtime.matrix(tensors["table"][:, offset:offset + self.size].contiguous())
         self.gate = runtime.matrix(tensors["gate.weight"])
-        self.proj = runtime.matrix(tensors["proj.weight"].t().contiguous())     # [size, hidden]: rows are read along the stream
+        self.proj_rows = runtime.matrix(tensors["proj.weight"])                 # [hidden, size], as a product takes it
+        self.proj = self.proj_rows.t().contiguous()                             # [size, hidden]: rows are read along the stream
         self.norm = runtime.vector(tensors["norm.weight"])
 
 

@@ -97,7 +97,8 @@ def project(x, weight, status, out_dtype=None, allow_partial=True):
 
 
 def paged_attention_generic(q, k_cache, v_cache, block_table, seq_of_token, positions, out, scale, window, status,
-                            chunk=None, softcap=None, keep_first=0, values_in_keys=None, sink=None, gate=None):
+                            chunk=None, softcap=None, keep_first=0, values_in_keys=None, sink=None, gate=None,
+                            value_gate=None):
     tokens, num_heads, head_size = q.shape
     _, num_kv_heads, page_size, _ = k_cache.shape
     groups = num_heads // num_kv_heads
@@ -123,6 +124,8 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, seq_of_token, posi
             scores = torch.cat([scores, sink.float()[:, None]], dim=1)
         probabilities = torch.softmax(scores, dim=-1)[:, :keys.shape[0]]
         mixed = torch.einsum("hn,nhd->hd", probabilities, v)
+        if value_gate is not None:      # logits, one per element of the mixed heads
+            mixed = mixed * torch.sigmoid(value_gate[t].float().reshape(mixed.shape))
         out[t] = (mixed if gate is None else gate[t][:, None] * mixed).to(out.dtype)
 
 
@@ -303,10 +306,12 @@ def per_head_project(x, weight, out):
 
 
 def router_topk(logits, top_k, score, renormalise, expert_ids, weights, num_experts=None, correction=None,
-                groups=None, group_best=1, renormalise_eps=0.0, weight_scale=1.0):
+                groups=None, group_best=1, renormalise_eps=0.0, weight_scale=1.0, bias=None):
     z = _summed(logits)
     if num_experts is not None:
         z = z[:, :num_experts]
+    if bias is not None:
+        z = z + bias
     scores = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, dim=-1)
     # without a correction the choice goes by the logits themselves (the scores are monotone in them)
     choice = z if correction is None else scores + correction
@@ -417,6 +422,31 @@ def conv_silu(x, weight, bias, conv_state, seq_of_token, q_start, state_slots, o
         decay_out.copy_(torch.exp(-torch.exp(a_log) * dt))
 
 
+def gate_in_place(qkv, channels, dtype):
+    return qkv.dim() == 2 and qkv.dtype == dtype
+
+
+def qkv_conv_store(qkv, bias, conv_weight, conv_state, seq_of_token, q_start, state_slots, slots, q_out, k_cache, v_cache,
+                   num_heads, num_kv_heads, key_size, value_size, status, positions=None, inv_freq=None, interleaved=False,
+                   gate_out=None, single_tokens=False):
+    channels = (num_heads + num_kv_heads) * key_size + num_kv_heads * value_size
+    values = _summed(qkv)
+    if gate_out is not None:
+        gate_out.copy_(values[:, channels:].to(gate_out.dtype))
+    values = values[:, :channels]
+    if bias is not None:
+        values = values + bias
+    if conv_weight is not None:
+        conv = torch.empty_like(values)
+        state = conv_state
+        if state is None:
+            state = torch.zeros((int(state_slots.max()) + 1, conv_weight.shape[1] - 1, channels), device=values.device)
+        conv_silu(values, conv_weight, None, state, seq_of_token, q_start, state_slots, conv, activation=False)
+        values = conv
+    qkv_norm_store(values, None, slots, q_out, k_cache, v_cache, num_heads, num_kv_heads, key_size, value_size, None,
+                   status, positions=positions, inv_freq=inv_freq, interleaved=interleaved)
+
+
 def linear_recurrence(q, k, v, state, q_start, state_slots, y, heads, groups, dim, vdim, head_decay=None,
                       token_decay=None, token_scale=None, skip=None, silu_inputs=False, max_q_len=None, rows=0,
                       segment_len=None, columns=0):
@@ -517,20 +547,27 @@ def _gelu_tanh(z):
     return 0.5 * z * (1.0 + torch.tanh(0.7978845608028654 * (z + 0.044715 * z ** 3)))
 
 
-def act_mul(gate_up, out, kind):
+def act_mul(gate_up, out, kind, limit=0.0, slope=1.0, up_shift=0.0):
     g = _summed(gate_up)
     inter = out.shape[1]
     gate, up = g[:, :inter], g[:, inter:]
+    if kind == "clamped_swish":
+        gate, up = torch.clamp(gate, max=limit), torch.clamp(up, min=-limit, max=limit)
+        out.copy_((gate / (1 + torch.exp(-slope * gate)) * (up + up_shift)).to(out.dtype))
+        return
     act = {"silu": lambda z: z / (1 + torch.exp(-z)), "gelu_tanh": _gelu_tanh}[kind]
     out.copy_((act(gate) * up).to(out.dtype))
 
 
-def _add_pending(residual, pending, scale):
+def _add_pending(residual, pending, scale, norm=None):
     terms = [t for t in (pending or []) if t is not None]
     if terms:
         total = _summed(terms[0])
         for t in terms[1:]:
             total = total + _summed(t)
+        if norm is not None:
+            weight, eps = norm
+            total = total * torch.rsqrt(total.pow(2).mean(-1, keepdim=True) + eps) * weight
         residual.add_(scale * total)
 
 
@@ -555,8 +592,22 @@ def norm_conv(pending, pending_scale, residual, norm_weight, eps, conv_weight, c
             conv_state[slot] = line[-(taps - 1):]
 
 
-def stream_tail(residual, pending, pending_scale, token_ids, side, depth):
-    _add_pending(residual, pending, pending_scale)
+def stream_norm(pending, pending_scale, pending_norm, residual, norm, out):
+    _add_pending(residual, pending, pending_scale, pending_norm)
+    if out is not None:
+        h = residual
+        if norm is not None:
+            weight, eps = norm
+            h = h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + eps) * weight
+        out.copy_(h.to(out.dtype))
+
+
+def side_gate(product, table, token_ids, out):
+    out.copy_((_gelu_tanh(_summed(product)) * table[token_ids.long()].float()).to(out.dtype))
+
+
+def stream_tail(residual, pending, pending_scale, token_ids, side, depth, pending_norm=None):
+    _add_pending(residual, pending, pending_scale, pending_norm)
     if side is not None:
         table, gate, proj_t, norm, eps = side
         g = _gelu_tanh(residual @ gate.float().T) * table[token_ids.long()].float()
@@ -709,7 +760,7 @@ _NAMES = (
     "moe_dispatch", "moe_gemm", "moe_combine", "softcap", "latent_decode_attention", "latent_decode_splits", "moe_gemm_on_tensor_cores", "moe_gemm_splits",
     "act_mul", "norm_conv", "stream_tail", "paged_attention_mixed", "gated_scan", "memory_gates", "memory_output",
     "norm_join", "memory_value_columns", "recurrence_step_splits", "latent_qkv_store", "hyper_norm",
-    "has_latent_attention",
+    "has_latent_attention", "stream_norm", "side_gate", "gate_in_place", "qkv_conv_store",
 )
 
 
