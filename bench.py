@@ -1711,6 +1711,237 @@ def latent_attention_points(name: str, heads: int, rate, status, out: dict) -> N
             del k
 
 
+def pugadra_sizes(width: int, heads: int, kv_heads: int, size: int, ff: int, vocab: int, window: int, layers: int) -> dict:
+    """A Pugadra configuration at the layer sizes of a Qwen2 model: windowed attention with convolutions of four
+    taps, every second layer reads the pages of the one before it; dense and routed feed-forwards in turn
+    (two of eight experts and a shared one, together as wide as the dense feed-forward), a token input of 64
+    values."""
+    def mixer(index):
+        m = {"heads": heads, "kv_heads": kv_heads, "dim": size, "vdim": size, "conv": 4, "scale": size ** -0.5,
+             "mask": {"size": window}, "rot": {"base": 1e6, "dims": size}}
+        return dict(m, kv_from=index - 1) if index % 2 else m
+
+    expert = ff // 3 // 8 * 8
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": expert, "limit": 7.0}, "router": {"experts": 8, "top": 2},
+           "shared": {"ff": expert, "limit": 7.0}}
+    return {"architecture": "Pugadra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "token_side": {"dim": 64},
+            "layers": [{"type": "attention", "mixer": mixer(i), "mlp": (dense, moe)[i % 2]} for i in range(layers)]}
+
+
+def run_pugadra(args) -> dict:
+    """Prefill and decode throughput of the Pugadra design at the layer sizes of the 0.5B and 1.5B models
+    (random weights, eight layers unless --layers says otherwise), beside Rekodra, the closest of the other
+    designs (attention with a sink, routed feed-forwards with a shared expert), and Qwen2, each with eight
+    layers at the same width, heads and vocabulary; then the design's own kernels alone, each beside its like."""
+    import torch
+
+    from einf_b200.cache import CacheManager
+    from einf_b200.config import EngineConfig, config_from_dict
+    from einf_b200.engine import ModelRunner
+    from einf_b200.sampling import Sampler
+
+    layers = args.layers or 8
+    result = {"scenario": "pugadra", "layers": layers, "context": CONTEXT, "window": 1024}
+    shapes = {"0.5b": (896, 4864, 14, 2, 64), "1.5b": (1536, 8960, 12, 2, 128)}
+    if args.only != "all":          # one small workload for a launch list
+        shapes = {"0.5b": shapes["0.5b"]}
+    for name, (width, ff, heads, kv_heads, size) in shapes.items():
+        qwen = dict(SIZES["1.5b"] if name == "1.5b" else QWEN25_05B, num_hidden_layers=layers, tie_word_embeddings=True)
+        vocab = qwen["vocab_size"]
+        ours = pugadra_sizes(width, heads, kv_heads, size, ff, vocab, 1024, layers)
+        near = rekodra_sizes(width, heads, kv_heads, size, ff, vocab, 1024)
+        for arch, cfg in (("pugadra", ours), ("rekodra", near), ("qwen2", qwen)):
+            if arch != "pugadra" and args.only != "all":
+                continue
+            pages = 64 * (CONTEXT // PAGE + 2) + 64
+            runner = ModelRunner.from_random(
+                config_from_dict(cfg), 0,
+                EngineConfig(dtype="bfloat16", block_len=PAGE, num_blocks=pages, max_batch_len=8192,
+                             max_prefill_chunk_len=8192, max_requests=64, use_cuda_graphs=not args.no_graphs))
+            manager = CacheManager(runner.group_specs(), runner.num_state_slots)
+            sampler = Sampler(runner.runtime.device, 64)
+            for tokens in {"decode": (), "prefill": (2048,)}.get(args.only, (2048, 8192)):
+                timed = time_prefill(runner, sampler, manager, tokens, repeats=2 if args.only == "prefill" else 5)
+                result[f"{name}_{arch}_prefill{tokens}_ms"] = round(timed["ms"], 3)
+                result[f"{name}_{arch}_prefill{tokens}_tokens_per_s"] = round(tokens / (timed["ms"] * 1e-3))
+            for batch in {"decode": (args.batch,), "prefill": ()}.get(args.only, (1, 8, 64)):
+                timed = time_decode(runner, sampler, manager, batch, CONTEXT, args.steps, args.warmup,
+                                    min_seconds=0.0 if args.only == "decode" else 0.2)
+                result[f"{name}_{arch}_decode_b{batch}_ms"] = round(timed["ms_per_step"], 3)
+                result[f"{name}_{arch}_decode_b{batch}_tokens_per_s"] = round(timed["tokens_per_s"], 1)
+                result[f"{name}_{arch}_decode_b{batch}_launches_per_step"] = timed["launches"] // max(1, args.steps)
+            del runner, manager, sampler
+            torch.cuda.empty_cache()
+    if args.only not in ("decode", "prefill"):
+        result["kernels"] = pugadra_kernels(peaks())
+    return result
+
+
+def pugadra_kernels(peak: dict) -> dict:
+    """The design's kernels alone (microseconds per launch in a CUDA graph of launches on rotating buffers
+    larger than the L2) with the bytes or flops each must move, each beside the like kernel of another
+    path: windowed attention with a sink and a gate per element beside the same without, the store kernel
+    with its convolution beside the rotary store of Qwen2, the norms behind and in front of a sublayer beside
+    the residual norm, the end of a layer in one kernel and as two products, the clamped gate beside SiLU's,
+    the router with a bias beside the plain one."""
+    import torch
+
+    from einf_b200 import ops
+
+    device = torch.device("cuda:0")
+    status = torch.zeros(1, dtype=torch.int32, device=device)
+    out: dict = {}
+    gbs, tflops = peak["hbm_gbs"], peak["bf16_tflops"]
+    turn = [0]
+
+    def rate(key, us, nbytes=0, flops=0):
+        out[key + "_us"] = round(us, 1)
+        if nbytes:
+            out[key + "_hbm_frac"] = round(nbytes / us / 1e3 / gbs, 3)
+        if flops:
+            out[key + "_flops_frac"] = round(flops / us / 1e6 / tflops, 4)
+
+    def timed(key, fn, make, bytes_each, nbytes=0, flops=0):
+        buffers = [make() for _ in range(max(2, min(64, int(300e6 / bytes_each))))]
+
+        def call():
+            turn[0] += 1
+            fn(buffers[turn[0] % len(buffers)])
+
+        rate(key, _graph_time_us(call, max(8, len(buffers))), nbytes, flops)
+
+    window, taps = 1024, 4
+    for name, width, ff, heads, kv_heads, size in (("0.5b", 896, 4864, 14, 2, 64), ("1.5b", 1536, 8960, 12, 2, 128)):
+        ops.ensure_built(list(ops.attention_libraries(size, PAGE)) + ["pointwise", "stream", "qkv_conv", "routed", "gemm_tcgen05"])
+        sink = torch.zeros(heads, device=device)
+        # --- attention: a prompt of 2,048 tokens, single tokens of 8 and 64 requests at 4,096
+        tokens, launches = 2048, 8
+        pages = tokens // PAGE
+        k = torch.randn(pages * launches + 4, kv_heads, PAGE, size, device=device).bfloat16()
+        v = torch.randn_like(k)
+        q = torch.randn(tokens, heads, size, device=device).bfloat16()
+        o = torch.empty_like(q)
+        product = torch.randn(tokens, (2 * heads + 2 * kv_heads) * size, device=device).bfloat16()
+        logits = product[:, (heads + 2 * kv_heads) * size:]
+        tables = [torch.arange(i * pages, (i + 1) * pages, dtype=torch.int32, device=device).view(1, -1) for i in range(launches)]
+        tiles = torch.tensor([[0, first, 128, first] for first in range(0, tokens, 128)], dtype=torch.int32, device=device)
+        flops = 4 * heads * size * sum(min(i + 1, window) for i in range(tokens))
+        for what, s, g in (("window", None, None), ("window_sink", sink, None), ("window_sink_gate", sink, logits)):
+            def prefill():
+                turn[0] += 1
+                ops.paged_prefill_attention(q, k, v, tables[turn[0] % launches], tiles, o, size ** -0.5, window, status,
+                                            cached_before=0, sink=s, value_gate=g)
+
+            rate(f"{name}_prefill2048_attention_{what}", _graph_time_us(prefill, launches), flops=flops)
+        del k, v
+        for batch in (8, 64):
+            pages = CONTEXT // PAGE
+            k = torch.randn(pages * batch * launches + 2, kv_heads, PAGE, size, device=device).bfloat16()
+            v = torch.randn_like(k)
+            qd = torch.randn(batch, heads, size, device=device).bfloat16()
+            od = torch.empty_like(qd)
+            gate = torch.randn(batch, heads * size, device=device).bfloat16()
+            dtables = [torch.arange(i * pages * batch, (i + 1) * pages * batch, dtype=torch.int32, device=device).view(batch, pages)
+                       for i in range(launches)]
+            seq = torch.arange(batch, dtype=torch.int32, device=device)
+            positions = torch.full((batch,), CONTEXT - 1, dtype=torch.int32, device=device)
+            for what, s, g in (("window", None, None), ("window_sink_gate", sink, gate)):
+                def decode():
+                    turn[0] += 1
+                    ops.paged_decode_attention_auto(qd, k, v, dtables[turn[0] % launches], seq, positions, od, size ** -0.5,
+                                                    window, status, max_context=CONTEXT, sink=s, value_gate=g)
+
+                rate(f"{name}_decode_b{batch}_attention_{what}", _graph_time_us(decode, launches),
+                     nbytes=2 * batch * window * kv_heads * size * 2)
+            del k, v
+        # --- everything between the products: a prompt of 2,048 tokens, single tokens of 8 and 64 requests
+        channels, gated = (heads + 2 * kv_heads) * size, heads * size
+        inv_freq = (1e6 ** (-torch.arange(size // 2, device=device).float() / (size // 2))).contiguous()
+        bias, taps_w = torch.randn(channels, device=device), torch.randn(channels, taps, device=device)
+        weight = torch.ones(width, device=device)
+        side = 64
+        table = torch.randn(4096, side, device=device).bfloat16()
+        gate_w, proj = torch.randn(side, width, device=device).bfloat16() * 0.03, torch.randn(width, side, device=device).bfloat16()
+        proj_t = proj.t().contiguous()
+        for what, lengths, splits in (("prompt2048", [2048], 1), ("decode_b8", [1] * 8, 8), ("decode_b64", [1] * 64, 8)):
+            requests, rows = len(lengths), sum(lengths)
+            starts = torch.tensor([0] + list(torch.tensor(lengths).cumsum(0)), dtype=torch.int32, device=device)
+            slots = torch.arange(rows, dtype=torch.int32, device=device)
+            state_slots = torch.arange(requests, dtype=torch.int32, device=device)
+            seq = torch.repeat_interleave(torch.arange(requests, device=device), torch.tensor(lengths, device=device)).to(torch.int32)
+            positions = torch.arange(rows, dtype=torch.int32, device=device)
+            k = torch.zeros(rows // PAGE + 2, kv_heads, PAGE, size, device=device).bfloat16()
+            v = torch.zeros_like(k)
+            singles = rows == requests
+            element = 4 * splits if splits > 1 else 2
+
+            def rows_of(columns):
+                return torch.randn(splits, rows, columns, device=device) if splits > 1 else \
+                    torch.randn(rows, columns, device=device).bfloat16()
+
+            def make_store():
+                return (rows_of(channels + gated), torch.empty(rows, heads, size, device=device).bfloat16(),
+                        torch.empty(rows, gated, device=device).bfloat16(),
+                        torch.zeros(requests, taps - 1, channels, device=device))
+
+            moved = rows * (channels + (gated if splits > 1 else 0)) * (element + 2) + 2 * requests * (taps - 1) * channels * 4
+            timed(f"{name}_{what}_store_convolved",
+                  lambda b: ops.qkv_conv_store(b[0], bias, taps_w, b[3], seq, starts, state_slots, slots, b[1], k, v, heads,
+                                               kv_heads, size, size, status, positions=positions, inv_freq=inv_freq,
+                                               interleaved=True, gate_out=b[2] if splits > 1 else None, single_tokens=singles),
+                  make_store, rows * (channels + gated) * element, nbytes=moved)
+            timed(f"{name}_{what}_store_rotary_qwen2",
+                  lambda b: ops.rope_kv_write(b[0], bias, positions, inv_freq, slots, b[1], k, v, heads, kv_heads, size, status),
+                  lambda: (rows_of(channels), torch.empty(rows, heads, size, device=device).bfloat16()),
+                  rows * channels * element, nbytes=rows * channels * (element + 2))
+
+            def make_norm():
+                return (rows_of(width), torch.randn(rows, width, device=device), torch.empty(rows, width, device=device).bfloat16())
+
+            nbytes = rows * width * (element + 8 + 2)
+            timed(f"{name}_{what}_norm_behind_and_ahead",
+                  lambda b: ops.stream_norm([b[0]], 0.5, (weight, 1e-6), b[1], (weight, 1e-6), b[2]), make_norm, nbytes,
+                  nbytes=nbytes)
+            timed(f"{name}_{what}_residual_norm",
+                  lambda b: ops.add_rmsnorm(b[0], b[1], weight, 1e-6, b[2], None, status), make_norm, nbytes, nbytes=nbytes)
+            # the end of a layer
+            ids = torch.randint(0, 4096, (rows,), device=device, dtype=torch.int32)
+
+            def as_products(b):
+                ops.stream_norm([b[0]], 0.5, (weight, 1e-6), b[1], None, b[2])
+                s = ops.project(b[2], gate_w, status)
+                ops.side_gate(s, table, ids, b[3])
+                y = ops.project(b[3], proj, status)
+                ops.stream_norm([y], 0.5, (weight, 1e-6), b[1], (weight, 1e-6), b[2])      # the next layer's first norm too
+
+            def make_tail():
+                return (*make_norm(), torch.empty(rows, side, device=device).bfloat16())
+
+            nbytes = rows * width * (element + 8)
+            timed(f"{name}_{what}_end_of_layer_products", as_products, make_tail, nbytes, nbytes=nbytes)
+            timed(f"{name}_{what}_end_of_layer_one_kernel",
+                  lambda b: ops.stream_tail(b[1], [b[0]], 0.5, ids, (table, gate_w, proj_t, weight, 1e-6), None), make_tail,
+                  nbytes, nbytes=nbytes)
+            nbytes = rows * ff * (2 * element + 2)
+
+            def make_gate():
+                return rows_of(2 * ff), torch.empty(rows, ff, device=device).bfloat16()
+
+            timed(f"{name}_{what}_clamped_gate",
+                  lambda b: ops.act_mul(b[0], b[1], "clamped_swish", limit=7.0, slope=1.702, up_shift=1.0), make_gate, nbytes,
+                  nbytes=nbytes)
+            timed(f"{name}_{what}_silu_gate", lambda b: ops.silu_mul(b[0], b[1]), make_gate, nbytes, nbytes=nbytes)
+            scores, router_bias = torch.randn(rows, 8, device=device), torch.randn(8, device=device)
+            chosen, shares = torch.empty(rows, 2, dtype=torch.int32, device=device), torch.empty(rows, 2, device=device)
+            for kind, extra in (("bias", router_bias), ("plain", None)):
+                rate(f"{name}_{what}_router_{kind}", _graph_time_us(
+                    lambda: ops.router_topk(scores, 2, "softmax", True, chosen, shares, bias=extra), 8))
+    out["status"] = int(status)
+    return out
+
+
 def run_decode_sizes(args) -> dict:
     """Decode at the 1.5B and 7B sizes of the family (batch 8 and 64, context 4,096) with the
     fraction of the HBM roofline each step reaches: at these sizes a step's kernels are long
@@ -2047,7 +2278,7 @@ def main() -> int:
                         help="leave the 1.5B and 7B workloads out of `points` (they take about a minute)")
     parser.add_argument("--lookahead", type=int, default=8,
                         help="EngineConfig.decode_lookahead of the end-to-end run: decode steps per report to the host")
-    parser.add_argument("--scenario", choices=("default", "1.5b-mixed", "7b-preempt", "decode-sizes", "decode-contexts", "sampling", "prefill-attention", "decode-attention", "prefill-sizes", "tepavik", "bomipel", "bomipel-kernels", "kanavik", "kanavik-kernels", "rekodra", "rekodra-kernels", "sorizen", "sorizen-kernels"), default="default",
+    parser.add_argument("--scenario", choices=("default", "1.5b-mixed", "7b-preempt", "decode-sizes", "decode-contexts", "sampling", "prefill-attention", "decode-attention", "prefill-sizes", "tepavik", "bomipel", "bomipel-kernels", "kanavik", "kanavik-kernels", "rekodra", "rekodra-kernels", "sorizen", "sorizen-kernels", "pugadra", "pugadra-kernels"), default="default",
                         help="other workloads of the baseline: a mixed step at 1.5B sizes, decoding under "
                              "cache pressure at 7B sizes, decode rooflines at 1.5B and 7B sizes; each prints "
                              "its own JSON line")
@@ -2085,7 +2316,8 @@ def main() -> int:
         return 0
     scenarios = {"1.5b-mixed": run_mixed_15b, "7b-preempt": run_preempt_7b, "decode-sizes": run_decode_sizes, "decode-contexts": run_decode_contexts, "decode-attention": run_decode_attention, "prefill-sizes": run_prefill_sizes, "tepavik": run_tepavik, "bomipel": run_bomipel, "kanavik": run_kanavik,
                  "kanavik-kernels": lambda args: {"scenario": "kanavik-kernels", "kernels": kanavik_kernels(peaks())},
-                 "rekodra": run_rekodra, "sorizen": run_sorizen,
+                 "rekodra": run_rekodra, "sorizen": run_sorizen, "pugadra": run_pugadra,
+                 "pugadra-kernels": lambda args: {"scenario": "pugadra-kernels", "kernels": pugadra_kernels(peaks())},
                  "sorizen-kernels": lambda args: {"scenario": "sorizen-kernels", "kernels": sorizen_kernels(peaks())},
                  "rekodra-kernels": lambda args: {"scenario": "rekodra-kernels", "kernels": rekodra_kernels(peaks())},
                  "bomipel-kernels": lambda args: {"scenario": "bomipel-kernels", "kernels": bomipel_kernels(peaks())},

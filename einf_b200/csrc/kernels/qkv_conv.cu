@@ -160,46 +160,78 @@ __global__ void qkv_conv_head_kernel(const TIn* __restrict__ qkv, const __grid_c
 
 // ---------------------------------------------------------------------------
 // Prompt sizes: bfloat16 rows, pairs interleaved (or no rotation), everything in whole pieces of eight
-// elements.  A thread has one piece of the row for kRun consecutive tokens: it reads every row's piece
-// once (16 bytes) and carries the taps - 1 inputs before it in registers; where a request starts it
-// takes them from the request's state.  The run's angles are made once per CTA.
+// elements.  A thread has one piece of the row for a run of consecutive tokens: it reads every row's
+// piece once (16 bytes) and carries the taps - 1 inputs before it in registers; where a request starts it
+// takes them from the request's state.  The first taps - 1 tokens of a request, the only ones that see
+// the state, all belong to the run in which the request starts (a run may so reach up to taps - 2 tokens
+// beyond its end, and the next one leaves them out); the thread that has read the state there moves it
+// on in the same breath, since the request's last inputs are rows of the product.  The run's angles,
+// requests and cache places are made once per CTA, from the step's inputs alone, while the product
+// before this kernel still runs.
 // ---------------------------------------------------------------------------
-constexpr int kRun = 8;
-constexpr int kPieceThreads = 128;
+constexpr int kRun = 8;                  // rows whose loads are in flight together
+constexpr int kPieceThreads = 256;       // at most
 
 template <int kTaps>
-__global__ void __launch_bounds__(kPieceThreads)
+__global__ void __launch_bounds__(kPieceThreads, 2)
 qkv_conv_piece_kernel(const __nv_bfloat16* __restrict__ qkv, const __grid_constant__ ConvStore p,
                       __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_cache,
                       __nv_bfloat16* __restrict__ v_cache) {
-  extern __shared__ float2 angles[];     // [kRun][pairs]: cosine, sine
+  constexpr int kKeep = kTaps - 1, kExtra = kKeep > 1 ? kKeep - 1 : 0;
+  extern __shared__ float2 angles[];     // [kRun + kExtra][pairs]: cosine, sine
+  // request_of: -1 for a token of another run
+  __shared__ int request_of[kRun + kExtra], first_of[kRun + kExtra], page_of[kRun + kExtra], offset_of[kRun + kExtra];
   pdl_launch_dependents();
-  const int t0 = blockIdx.y * kRun, count = min(kRun, p.num_tokens - t0);
-  for (int i = threadIdx.x; i < count * p.pairs; i += kPieceThreads) {
+  const int t0 = blockIdx.y * kRun, count = min(kRun + kExtra, p.num_tokens - t0);
+  for (int s = threadIdx.x; s < count; s += blockDim.x) {
+    const int t = t0 + s, r = p.seq_of_token[t], first = p.q_start[r];
+    const bool sees_state = t - first < kKeep;
+    const bool mine = s < kRun ? !sees_state || first >= t0 : sees_state && first < t0 + kRun;
+    request_of[s] = mine ? r : -1;
+    first_of[s] = first;
+    int page = 0, offset = 0;
+    page_of[s] = cache_place(p, t, page, offset, false) ? page : -1;
+    offset_of[s] = offset;
+  }
+  for (int i = threadIdx.x; i < count * p.pairs; i += blockDim.x) {
     const int s = i / p.pairs, pair = i - s * p.pairs;
     float sn, cs;
-    sincosf((float)p.positions[t0 + s] * p.inv_freq[pair], &sn, &cs);     // inputs of the step
+    sincosf((float)p.positions[t0 + s] * p.inv_freq[pair], &sn, &cs);
     angles[i] = make_float2(cs, sn);
+  }
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  const bool live = c < p.channels;
+  float w[kTaps][8], bias[8];            // weights: no kernel of the step writes them
+  if (live) {
+#pragma unroll
+    for (int e = 0; e < 8; e += 4) {
+      const float4 b = p.bias ? *reinterpret_cast<const float4*>(p.bias + c + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+      bias[e] = b.x; bias[e + 1] = b.y; bias[e + 2] = b.z; bias[e + 3] = b.w;
+    }
+    // the taps of eight channels lie one after the other: whole float4s
+#pragma unroll
+    for (int i = 0; i < 2 * kTaps; ++i) {
+      const float4 v = p.weight ? *reinterpret_cast<const float4*>(p.weight + (size_t)c * kTaps + 4 * i)
+                                : make_float4(1.f, 1.f, 1.f, 1.f);
+      const float part[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) w[(4 * i + j) % kTaps][(4 * i + j) / kTaps] = part[j];
+    }
   }
   __syncthreads();
   pdl_wait();
-  const int c = (blockIdx.x * kPieceThreads + threadIdx.x) * 8;
-  if (c >= p.channels) return;
+  if (p.slots && blockIdx.x == 0 && threadIdx.x < count && page_of[threadIdx.x] < 0 && p.slots[t0 + threadIdx.x] >= 0)
+    atomicOr(p.status, kStatusBadPage);
+  if (!live) return;
   const int queries = p.num_heads * p.key_size, keys = p.num_kv_heads * p.key_size;
   const bool is_query = c < queries, is_value = c >= queries + keys;
   const int local = is_query ? c : (is_value ? c - queries - keys : c - queries);
   const int size = is_value ? p.value_size : p.key_size;
   const int head = local / size, d = local - head * size;
   const bool rotates = !is_value && d < 2 * p.pairs;
-  constexpr int kKeep = kTaps - 1;
 
-  float w[kTaps][8], bias[8], past[kKeep > 0 ? kKeep : 1][8];
-#pragma unroll
-  for (int e = 0; e < 8; ++e) {
-    bias[e] = p.bias ? p.bias[c + e] : 0.f;
-#pragma unroll
-    for (int j = 0; j < kTaps; ++j) w[j][e] = p.weight ? p.weight[(size_t)(c + e) * kTaps + j] : 1.f;
-  }
+  float past[kKeep > 0 ? kKeep : 1][8];
+  auto load_row = [&](int t) { return *reinterpret_cast<const uint4*>(qkv + (size_t)t * p.width + c); };
   auto unpack = [&](const uint4& raw, float (&u)[8]) {
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
@@ -209,74 +241,96 @@ qkv_conv_piece_kernel(const __nv_bfloat16* __restrict__ qkv, const __grid_consta
       u[2 * e + 1] = f.y + bias[2 * e + 1];
     }
   };
-  uint4 raw[kRun];
+  // The inputs before token t of request r: rows of the step, or, for the request's first token, its state, whose
+  // place then gets the request's last inputs (a portion shorter than that keeps the tail of the old ones in front).
+  auto enter = [&](int t, int r, int first) {
+    if (t > first) {                     // the run starts inside the request, where no token sees the state
 #pragma unroll
-  for (int s = 0; s < kRun; ++s)
-    raw[s] = *reinterpret_cast<const uint4*>(qkv + (size_t)(t0 + min(s, count - 1)) * p.width + c);
-  int request = -1;
+      for (int j = 0; j < kKeep; ++j) unpack(load_row(t - kKeep + j), past[j]);
+      return;
+    }
+    float* state = request_state(p, r);
 #pragma unroll
-  for (int s = 0; s < kRun; ++s) {
-    if (s < count) {
-      const int t = t0 + s, r = p.seq_of_token[t];
-      if (kKeep > 0 && r != request) {
-        // the inputs before this token: rows of the step, or the request's state ahead of its first token
-        const int first = p.q_start[r];
-        const float* state = request_state(p, r);
+    for (int j = 0; j < kKeep; ++j)
 #pragma unroll
-        for (int j = 0; j < kKeep; ++j) {
-          const int src = t - kKeep + j;
-          if (src >= first) {
-            unpack(*reinterpret_cast<const uint4*>(qkv + (size_t)src * p.width + c), past[j]);
-          } else {
-#pragma unroll
-            for (int e = 0; e < 8; ++e) past[j][e] = state ? state[(size_t)(kKeep - (first - src)) * p.channels + c + e] : 0.f;
-          }
-        }
-        request = r;
+      for (int e = 0; e < 8; e += 4) {
+        const float4 v = state ? *reinterpret_cast<const float4*>(state + (size_t)j * p.channels + c + e)
+                               : make_float4(0.f, 0.f, 0.f, 0.f);
+        past[j][e] = v.x; past[j][e + 1] = v.y; past[j][e + 2] = v.z; past[j][e + 3] = v.w;
       }
-      float u[8], y[8];
-      unpack(raw[s], u);
+    if (!state) return;
+    const int length = p.q_start[r + 1] - first;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        float acc = 0.f;
-#pragma unroll
-        for (int j = 0; j < kKeep; ++j) acc = fmaf(w[j][e], past[j][e], acc);
-        y[e] = fmaf(w[kKeep][e], u[e], acc);
-#pragma unroll
-        for (int j = 0; j + 1 < kKeep; ++j) past[j][e] = past[j + 1][e];
-        if (kKeep > 0) past[kKeep > 0 ? kKeep - 1 : 0][e] = u[e];
-      }
-      if (rotates) {
-        const float2* a = angles + s * p.pairs + (d >> 1);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float2 cs = a[e];
-          const float even = y[2 * e], odd = y[2 * e + 1];
-          y[2 * e] = even * cs.x - odd * cs.y;
-          y[2 * e + 1] = odd * cs.x + even * cs.y;
-        }
-      }
-      __nv_bfloat16* dst = nullptr;
-      if (is_query) {
-        dst = q_out + (size_t)t * queries + c;
-      } else {
-        int page = 0, offset = 0;
-        if (cache_place(p, t, page, offset, local == 0))
-          dst = (is_value ? v_cache : k_cache) + (((size_t)page * p.num_kv_heads + head) * p.page_size + offset) * size + d;
-      }
-      if (dst) {
-        uint4 packed;
-        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&packed);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(y[2 * e], y[2 * e + 1]);
-        *reinterpret_cast<uint4*>(dst) = packed;
+    for (int j = 0; j < kKeep; ++j) {
+      const int rel = length - kKeep + j;
+      float4* row = reinterpret_cast<float4*>(state + (size_t)j * p.channels + c);
+      if (rel >= 0) {
+        float fresh[8];
+        unpack(load_row(first + rel), fresh);
+        row[0] = make_float4(fresh[0], fresh[1], fresh[2], fresh[3]);
+        row[1] = make_float4(fresh[4], fresh[5], fresh[6], fresh[7]);
+      } else {                           // a later row, not yet written
+        const float4* old = reinterpret_cast<const float4*>(state + (size_t)(j + length) * p.channels + c);
+        row[0] = old[0];
+        row[1] = old[1];
       }
     }
-  }
+  };
+  int request = -1;
+  auto step = [&](int s, const uint4& raw) {
+    const int t = t0 + s, r = request_of[s];
+    if (r < 0) return;
+    if (kKeep > 0 && r != request) enter(t, r, first_of[s]);
+    request = r;
+    float u[8], y[8];
+    unpack(raw, u);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < kKeep; ++j) acc = fmaf(w[j][e], past[j][e], acc);
+      y[e] = fmaf(w[kKeep][e], u[e], acc);
+#pragma unroll
+      for (int j = 0; j + 1 < kKeep; ++j) past[j][e] = past[j + 1][e];
+      if (kKeep > 0) past[kKeep > 0 ? kKeep - 1 : 0][e] = u[e];
+    }
+    if (rotates) {
+      const float2* a = angles + s * p.pairs + (d >> 1);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 cs = a[e];
+        const float even = y[2 * e], odd = y[2 * e + 1];
+        y[2 * e] = even * cs.x - odd * cs.y;
+        y[2 * e + 1] = odd * cs.x + even * cs.y;
+      }
+    }
+    __nv_bfloat16* dst;
+    if (is_query) {
+      dst = q_out + (size_t)t * queries + c;
+    } else {
+      if (page_of[s] < 0) return;
+      dst = (is_value ? v_cache : k_cache) +
+            (((size_t)page_of[s] * p.num_kv_heads + head) * p.page_size + offset_of[s]) * size + d;
+    }
+    uint4 packed;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(y[2 * e], y[2 * e + 1]);
+    *reinterpret_cast<uint4*>(dst) = packed;
+  };
+  uint4 raw[kRun];
+#pragma unroll
+  for (int s = 0; s < kRun; ++s) raw[s] = load_row(t0 + min(s, count - 1));
+#pragma unroll
+  for (int s = 0; s < kRun; ++s)
+    if (s < count) step(s, raw[s]);
+#pragma unroll 1
+  for (int s = kRun; s < count; ++s)
+    if (request_of[s] >= 0) step(s, load_row(t0 + s));
 }
 
-// Afterwards a request's last taps - 1 inputs become its state (a portion shorter than that keeps the
-// tail of the old state in front).  One thread per (request, channel).
+// After the head-by-head kernel a request's last taps - 1 inputs become its state (a portion shorter than
+// that keeps the tail of the old state in front).  One thread per (request, channel).
 template <typename TIn>
 __global__ void qkv_conv_state_kernel(const TIn* __restrict__ qkv, const __grid_constant__ ConvStore p) {
   pdl_launch_dependents();
@@ -327,21 +381,28 @@ extern "C" int einf_qkv_conv_store(const void* qkv, int in_dtype, int splits, lo
                     single_tokens, status};
   const bool pieces = in_dtype == kBFloat16 && dtype == kBFloat16 && p.splits == 1 && !single_tokens && !gate_out &&
                       num_tokens >= 32 && taps <= 4 && key_size % 8 == 0 && value_size % 8 == 0 && width % 8 == 0 &&
-                      pairs % 4 == 0 && (interleaved || pairs == 0) && (num_tokens + kRun - 1) / kRun <= 65535 &&
-                      (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
+                      pairs % 4 == 0 && (interleaved || pairs == 0) && num_tokens <= 65535 * kRun &&
+                      (taps == 1 || state_stride % 4 == 0) &&
+                      (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)bias |
+                        (uintptr_t)conv_weight | (uintptr_t)conv_state) & 15) == 0;
   cudaError_t e = cudaSuccess;
   if (pieces) {
-    const dim3 grid((channels / 8 + kPieceThreads - 1) / kPieceThreads, (num_tokens + kRun - 1) / kRun);
-    const size_t smem = (size_t)kRun * pairs * sizeof(float2);
+    // equal shares of a row's pieces, so that few threads are left over
+    const int shares = (channels / 8 + kPieceThreads - 1) / kPieceThreads;
+    const int threads = ((channels / 8 + shares - 1) / shares + 31) / 32 * 32;
+    const dim3 grid(shares, (num_tokens + kRun - 1) / kRun);
 #define EINF_PIECES(TAPS)                                                                                        \
-  e = launch_pdl(qkv_conv_piece_kernel<TAPS>, grid, kPieceThreads, smem, stream, (const __nv_bfloat16*)qkv, p,   \
-                 (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache)
+  e = launch_pdl(qkv_conv_piece_kernel<TAPS>, grid, threads, (size_t)(kRun + TAPS) * pairs * sizeof(float2),     \
+                 stream, (const __nv_bfloat16*)qkv, p, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache,           \
+                 (__nv_bfloat16*)v_cache)
     if (taps == 1) EINF_PIECES(1);
     else if (taps == 2) EINF_PIECES(2);
     else if (taps == 3) EINF_PIECES(3);
     else EINF_PIECES(4);
 #undef EINF_PIECES
-  } else {
+    return (int)e;
+  }
+  {
     const int items = num_heads + 2 * num_kv_heads + (gate_out ? num_heads : 0);
     if (items > 65535) return (int)cudaErrorInvalidValue;
     const int largest = key_size > value_size ? key_size : value_size;

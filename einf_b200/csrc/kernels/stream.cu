@@ -355,7 +355,7 @@ __global__ void side_gate_kernel(const TIn* __restrict__ product, int splits, lo
 
 // ---------------------------------------------------------------------------
 // The end of a layer.  One CTA per token, the row x in shared memory:
-//   x = residual[t] + scale * pending[t]   (post != null: of its RMS norm, as above)
+//   x = residual[t] + scale * pending[t]
 //   token input (table != null):  s = gate x  [n];  g = gelu(s) * table[token]  [n];  y = proj_t^T g  [H];
 //                                 x += scale * y * rsqrt(mean(y^2) + eps) * norm
 //   depth average (history != null):  history[index + 1][t] = x;
@@ -370,7 +370,7 @@ __global__ void stream_tail_kernel(float* __restrict__ residual, const __grid_co
                                    const TW* __restrict__ gate, const TW* __restrict__ proj_t,
                                    const float* __restrict__ norm, int side, int vocab, float eps,
                                    float* __restrict__ history, int depth_index, const float* __restrict__ depth_weight,
-                                   long long history_stride, const float* __restrict__ post, float post_eps, int hidden) {
+                                   long long history_stride, int hidden) {
   extern __shared__ float smem[];
   float* x = smem;                   // [hidden]
   float* y = x + hidden;             // [hidden]
@@ -381,21 +381,10 @@ __global__ void stream_tail_kernel(float* __restrict__ residual, const __grid_co
   const int t = blockIdx.x;
   const size_t base = (size_t)t * hidden;
   const bool adds = pending.a != nullptr || pending.b != nullptr;
-  if (post && adds) {
-    float ss = 0.f;
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-      const float v = pending_sum(pending, base + c);
-      y[c] = v;
-      ss = fmaf(v, v, ss);
-    }
-    const float factor = scale * rsqrtf(block_sum(ss, red) / (float)hidden + post_eps);
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) x[c] = fmaf(factor * post[c], y[c], residual[base + c]);
-  } else {
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-      float v = residual[base + c];
-      if (adds) v += scale * pending_sum(pending, base + c);
-      x[c] = v;
-    }
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    float v = residual[base + c];
+    if (adds) v += scale * pending_sum(pending, base + c);
+    x[c] = v;
   }
   __syncthreads();
   if (table) {
@@ -473,8 +462,7 @@ stream_tail_tokens_kernel(float* __restrict__ residual, const __grid_constant__ 
                           const int* __restrict__ token_ids, const TW* __restrict__ table, const TW* __restrict__ gate,
                           const TW* __restrict__ proj_t, const float* __restrict__ norm, int side, int vocab, float eps,
                           float* __restrict__ history, int depth_index, const float* __restrict__ depth_weight,
-                          long long history_stride, const float* __restrict__ post, float post_eps, int hidden,
-                          int num_tokens) {
+                          long long history_stride, int hidden, int num_tokens) {
   extern __shared__ float4 smem4[];
   float* x = (float*)smem4;          // [TB, hidden]
   float* y = x + TB * hidden;        // [TB, hidden]
@@ -487,40 +475,15 @@ stream_tail_tokens_kernel(float* __restrict__ residual, const __grid_constant__ 
   const int t0 = blockIdx.x * TB;
   const int count = min(TB, num_tokens - t0);
   const bool adds = pending.a != nullptr || pending.b != nullptr;
-  if (post && adds) {
-    // the pending rows and their sums of squares first; every thread reads back the columns it wrote itself
-#pragma unroll 1
-    for (int i = 0; i < TB; ++i) {
-      float ss = 0.f;
-      for (int c = tid; c < hidden; c += kTailThreads) {
-        const float v = i < count ? pending_sum(pending, (size_t)(t0 + i) * hidden + c) : 0.f;
-        y[i * hidden + c] = v;
-        ss = fmaf(v, v, ss);
-      }
-      ss = warp_sum(ss);
-      if (lane == 0) red[i * kWarps + warp] = ss;
+  for (int idx = tid; idx < TB * hidden; idx += kTailThreads) {
+    const int i = idx / hidden;
+    float v = 0.f;
+    if (i < count) {
+      const size_t at = (size_t)t0 * hidden + idx;
+      v = residual[at];
+      if (adds) v += scale * pending_sum(pending, at);
     }
-    __syncthreads();
-#pragma unroll 1
-    for (int i = 0; i < TB; ++i) {
-      float total = 0.f;
-#pragma unroll
-      for (int w = 0; w < kWarps; ++w) total += red[i * kWarps + w];
-      const float factor = scale * rsqrtf(total / (float)hidden + post_eps);
-      for (int c = tid; c < hidden; c += kTailThreads)
-        x[i * hidden + c] = i < count ? fmaf(factor * post[c], y[i * hidden + c], residual[(size_t)(t0 + i) * hidden + c]) : 0.f;
-    }
-  } else {
-    for (int idx = tid; idx < TB * hidden; idx += kTailThreads) {
-      const int i = idx / hidden;
-      float v = 0.f;
-      if (i < count) {
-        const size_t at = (size_t)t0 * hidden + idx;
-        v = residual[at];
-        if (adds) v += scale * pending_sum(pending, at);
-      }
-      x[idx] = v;
-    }
+    x[idx] = v;
   }
   __syncthreads();
   if (table) {
@@ -716,6 +679,7 @@ extern "C" int einf_stream_norm(const void* pend_a, int a_dtype, int a_splits, l
       if (num_tokens >= 256 && hidden <= 2048 && a_splits <= 1) {
         const int grid = (num_tokens + 7) / 8;
         if (hidden <= 1024) EINF_STREAM_NORM(32, 8, grid, 256);
+        if (hidden <= 1536) EINF_STREAM_NORM(32, 12, grid, 256);
         EINF_STREAM_NORM(32, 16, grid, 256);
       }
       if (hidden <= 512) EINF_STREAM_NORM(128, 1, num_tokens, 128);
@@ -756,8 +720,8 @@ extern "C" int einf_stream_tail(float* residual, const void* pend_a, int a_dtype
                                 const void* pend_b, int b_dtype, int b_splits, long long b_stride, float scale,
                                 const int* token_ids, const void* table, const void* gate, const void* proj_t,
                                 int weight_dtype, const float* norm, int side, int vocab, float eps, float* history,
-                                int depth_index, const float* depth_weight, long long history_stride,
-                                const float* post, float post_eps, int num_tokens, int hidden, cudaStream_t stream) {
+                                int depth_index, const float* depth_weight, long long history_stride, int num_tokens,
+                                int hidden, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (hidden <= 0 || side < 0) return (int)cudaErrorInvalidValue;
   const Pending pending{pend_a, a_dtype, a_splits, a_stride, pend_b, b_dtype, b_splits, b_stride};
@@ -777,7 +741,7 @@ extern "C" int einf_stream_tail(float* residual, const void* pend_a, int a_dtype
     }                                                                                                                   \
     return (int)launch_pdl(kernel, blocks, kTailThreads, bytes(TB), stream, residual, pending, scale, token_ids,       \
                            (const T*)table, (const T*)gate, (const T*)proj_t, norm, side, vocab, eps, history,          \
-                               depth_index, depth_weight, history_stride, post, post_eps, hidden, num_tokens);              \
+                           depth_index, depth_weight, history_stride, hidden, num_tokens);                              \
   })
       if (each == 8) EINF_TAIL(8)
       if (each == 1) EINF_TAIL(1)
@@ -794,6 +758,6 @@ extern "C" int einf_stream_tail(float* residual, const void* pend_a, int a_dtype
     }
     return (int)launch_pdl(stream_tail_kernel<T>, num_tokens, threads, smem, stream, residual, pending, scale,
                            token_ids, (const T*)table, (const T*)gate, (const T*)proj_t, norm, side, vocab, eps,
-                           history, depth_index, depth_weight, history_stride, post, post_eps, hidden);
+                           history, depth_index, depth_weight, history_stride, hidden);
   })
 }

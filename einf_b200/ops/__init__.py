@@ -962,8 +962,8 @@ def qkv_conv_store(
     biased inputs, oldest first; a view whose slot stride may be larger; not needed with one tap).  Rotation, ``slots``
     and the caches as in :func:`qkv_norm_store`, of the convolved values.  ``gate_out`` (q_out's dtype,
     ``[tokens, heads * value_size]``) receives the gate's columns.  ``single_tokens``: every request brings one
-    token, and one launch does it all; otherwise a second one moves the state on."""
-    global launch_count
+    token.  One launch does it all for those and for long steps of bfloat16 rows (up to four taps, sizes that are
+    multiples of eight); otherwise a second one moves the state on."""
     tokens, width = qkv.shape[-2:]
     channels = (num_heads + num_kv_heads) * key_size + num_kv_heads * value_size
     gated = num_heads * value_size
@@ -1030,8 +1030,6 @@ def qkv_conv_store(
            _stream()),
         "qkv_conv_store",
     )
-    if taps > 1 and not single_tokens:
-        launch_count += 1      # the state of the convolutions
 
 
 # ---------------------------------------------------------------------------
@@ -1956,11 +1954,9 @@ def stream_tail(
     token_ids: torch.Tensor,
     side: Optional[tuple],
     depth: Optional[tuple],
-    pending_norm: Optional[tuple] = None,
 ) -> None:
     """The end of a layer in one pass over every row of the stream, in 32-bit:
-    ``x = residual + pending_scale * sum(pending)`` (as in :func:`norm_conv`; with ``pending_norm`` through a norm, as
-    in :func:`stream_norm`); with ``side = (table
+    ``x = residual + pending_scale * sum(pending)`` (as in :func:`norm_conv`); with ``side = (table
     [vocab, n], gate [n, H], proj_t [n, H], norm [H] float32, eps)``: ``g = gelu(gate x) * table[token]``,
     ``y = proj_t^T g``, ``x += pending_scale * y * rsqrt(mean(y^2) + eps) * norm``; with ``depth =
     (history [L + 1, T, H] float32, index, weight [index + 2] float32)``: ``history[index + 1] = x`` and
@@ -1992,12 +1988,11 @@ def stream_tail(
         "einf_stream_tail",
         [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_longlong, c_float, c_void_p,
          c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_longlong,
-         c_void_p, c_float, c_int, c_int, c_void_p],
+         c_int, c_int, c_void_p],
     )
     _check(
         fn(_dev(residual, "residual"), *_pending_terms(pending, tokens, hidden), float(pending_scale),
-           _opt(token_ids, "token_ids", torch.int32), *side_args, *depth_args,
-           *_norm_constants(pending_norm, hidden, "pending_norm"), tokens, hidden, _stream()),
+           _opt(token_ids, "token_ids", torch.int32), *side_args, *depth_args, tokens, hidden, _stream()),
         "stream_tail",
     )
 

@@ -16,10 +16,13 @@ import torch
 
 from .. import ops
 from .base import CacheView, Part, StepContext, build_part, join_needs, part_class, register_part
+from .stream import NormedPending
 
 
 class Block(Part):
     mixer: Part
+    #: ``forward`` takes a :class:`~einf_b200.parts.stream.NormedPending` as what is pending
+    takes_normed_pending = False
 
     @classmethod
     def part_categories(cls) -> dict[str, str]:
@@ -107,17 +110,16 @@ class PreNormStreamBlock(Block):
     to the stream), a short causal convolution ``c(x) = x + conv(x)`` in front of a sublayer (run in the
     launch of the norm before it, continued from and into the request's state row), no feed-forward,
     a per-layer token input added after the feed-forward, and a weighted sum over the results of
-    all layers so far in place of the layer's own result.  The layer's last kernel adds the pending
-    sublayer output, the token input and the weighted sum in one pass over the row, so the block
-    hands nothing pending to the next one.  The block's state row holds the convolutions' inputs
-    in front of whatever state its mixer keeps."""
+    all layers so far in place of the layer's own result.  With a weighted sum the layer's last kernel
+    adds the pending sublayer output, the token input and the sum in one pass over the row, and the
+    block hands nothing pending to the next one; without one, what the layer added last stays pending
+    (:class:`~einf_b200.parts.stream.NormedPending`) until the next layer's first norm.  The block's
+    state row holds the convolutions' inputs in front of whatever state its mixer keeps."""
 
     optional_roles = ("mixer_conv", "mixer_post_norm", "feed_forward_norm", "feed_forward_conv", "feed_forward",
                       "feed_forward_post_norm", "token_input", "depth_mix")
 
-    #: from this many tokens on the token input's two matrices are products of their own instead of
-    #: part of the layer's last kernel
-    SIDE_PRODUCT_TOKENS = 128
+    takes_normed_pending = True
 
     @classmethod
     def part_categories(cls):
@@ -169,20 +171,20 @@ class PreNormStreamBlock(Block):
         rows = cache.state[:, offset:offset + (conv.taps - 1) * conv.size]
         return rows.unflatten(1, (conv.taps - 1, conv.size))
 
-    def _normalise(self, which: int, pending, post, residual, ctx, cache):
-        """Add what is pending (through the norm ``post`` behind its sublayer, if there is one) and return what
-        the next sublayer reads."""
+    def _normalise(self, which: int, pending, scale, post, residual, ctx, cache):
+        """Add ``scale`` times what is pending (through the norm ``post`` behind its sublayer, if there is one) and
+        return what the next sublayer reads."""
         norm = (self.mixer_norm, self.feed_forward_norm)[which]
         conv = (self.mixer_conv, self.feed_forward_conv)[which]
         out = torch.empty(residual.shape, dtype=self.runtime.dtype, device=residual.device)
         if conv is None:
-            ops.stream_norm(pending, self.residual_mult, self._constants(post), residual, self._constants(norm), out)
+            ops.stream_norm(pending, scale, post, residual, self._constants(norm), out)
             return out
         if pending is not None and post is not None:
-            ops.stream_norm(pending, self.residual_mult, self._constants(post), residual, None, None)
+            ops.stream_norm(pending, scale, post, residual, None, None)
             pending = None
         ops.norm_conv(
-            pending, self.residual_mult, residual, norm.weight, norm.eps, conv.weight,
+            pending, scale, residual, norm.weight, norm.eps, conv.weight,
             self._conv_state(which, cache), ctx.seq_of_token, ctx.q_start, ctx.state_slots, out,
             single_tokens=ctx.decode_only,
         )
@@ -193,45 +195,54 @@ class PreNormStreamBlock(Block):
         return None if norm is None else (norm.weight, norm.eps)
 
     def _add_token_input(self, terms, post, residual, ctx):
-        """The end of a layer at prompt sizes: the token input's two matrices on the tensor cores, between a
-        kernel that adds the pending output and one that adds the token input."""
+        """The token input's two matrices as products, behind a kernel that adds the pending output; the token
+        input itself stays pending."""
         side, tokens = self.token_input, residual.shape[0]
         x = torch.empty(residual.shape, dtype=self.runtime.dtype, device=residual.device)
-        ops.stream_norm(terms, self.residual_mult, self._constants(post), residual, None, x)
+        ops.stream_norm(terms, self.residual_mult, post, residual, None, x)
         product = ops.project(x, side.gate, ctx.status)
         g = torch.empty((tokens, side.size), dtype=self.runtime.dtype, device=residual.device)
         ops.side_gate(product, side.table, ctx.token_ids, g)
-        y = ops.project(g, side.proj_rows, ctx.status)
-        ops.stream_norm([y], self.residual_mult, (side.norm, side.eps), residual, None, None)
+        return NormedPending([ops.project(g, side.proj_rows, ctx.status)], self.residual_mult, (side.norm, side.eps))
 
     def forward(self, residual, pending, ctx, cache):
-        if pending is not None:
+        if pending is not None and not isinstance(pending, NormedPending):
             raise ValueError("a prenorm_stream layer follows one that left its output pending")
         depth = self.depth_mix
         history = None
         if depth is not None:
+            if pending is not None:
+                pending.settle(residual)
+                pending = None
             history = depth.history(ctx, residual)
             if depth.index == 0:
                 history[0].copy_(residual)      # the embedding output, before this layer changes the stream
-        x = self._normalise(0, None, None, residual, ctx, cache)
+        if pending is None:
+            x = self._normalise(0, None, 1.0, None, residual, ctx, cache)
+        else:
+            x = self._normalise(0, pending.terms, pending.scale, pending.norm, residual, ctx, cache)
         view = cache
         if self._mixer_offset is not None:
             view = CacheView(cache.group, cache.k, cache.v, cache.state[:, self._mixer_offset:], cache.writes,
                              cache.page_size)
         terms = self.mixer.forward_terms(x, ctx, view) if hasattr(self.mixer, "forward_terms") \
             else [self.mixer.forward(x, ctx, view)]
-        post = self.mixer_post_norm
+        post = self._constants(self.mixer_post_norm)
         if self.feed_forward is not None:
-            x = self._normalise(1, terms, post, residual, ctx, cache)
-            terms, post = [self.feed_forward.forward(x, ctx)], self.feed_forward_post_norm
+            x = self._normalise(1, terms, self.residual_mult, post, residual, ctx, cache)
+            terms, post = [self.feed_forward.forward(x, ctx)], self._constants(self.feed_forward_post_norm)
+        if depth is None:
+            if self.token_input is None:
+                return NormedPending(terms, self.residual_mult, post)
+            return self._add_token_input(terms, post, residual, ctx)
+        if post is not None:
+            ops.stream_norm(terms, self.residual_mult, post, residual, None, None)
+            terms = None
         side = self.token_input
-        if side is not None and depth is None and residual.shape[0] >= self.SIDE_PRODUCT_TOKENS:
-            self._add_token_input(terms, post, residual, ctx)
-            return None
         ops.stream_tail(
             residual, terms, self.residual_mult, ctx.token_ids,
             None if side is None else (side.table, side.gate, side.proj, side.norm, side.eps),
-            None if depth is None else (history, depth.index, depth.weight), pending_norm=self._constants(post),
+            (history, depth.index, depth.weight),
         )
         return None
 

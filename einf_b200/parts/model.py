@@ -17,7 +17,7 @@ from .base import (
     pages_of, state_of, walk_part_specs,
 )
 from .block import build_block
-from .stream import ResidualStreams
+from .stream import NormedPending, ResidualStreams
 
 
 def _part_specs(model_spec: ModelSpec):
@@ -150,6 +150,9 @@ class DecoderModel:
         first = residual.clone() if any(entry.add_embedding for entry in self.schedule) else None
         pending = None
         for index, entry in enumerate(self.schedule):
+            if isinstance(pending, NormedPending) and (entry.add_embedding or not self.blocks[entry.layer].takes_normed_pending):
+                pending.settle(residual)
+                pending = None
             if entry.add_embedding:
                 # one more float32 term of the pending output, which the entry's first norm adds up
                 terms = [first[None]]
@@ -157,6 +160,9 @@ class DecoderModel:
                     terms.insert(0, (pending if pending.dim() == 3 else pending[None]).to(torch.float32))
                 pending = torch.cat(terms, dim=0) if len(terms) > 1 else terms[0]
             pending = self.blocks[entry.layer].forward(residual, pending, ctx, caches[index])
+        if isinstance(pending, NormedPending):
+            pending.settle(residual)
+            pending = None
         if getattr(self.final_norm, "takes_status", False):
             x = self.final_norm.forward(pending, residual, rows=ctx.logit_rows, status=ctx.status)
         else:

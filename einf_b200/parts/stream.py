@@ -14,8 +14,9 @@ layer i is ``sum_(j <= i + 1) w[j] X_j``.  The results of all layers of the step
 32-bit buffer in ``ctx.extras``.
 
 The parts hold tensors and sizes; the block that arranges them (``prenorm_stream``) launches one
-kernel for the end of a layer: pending sublayer output, token input and weighted sum together (at prompt
-sizes without a weighted sum: two products with a kernel in front, between and behind).
+kernel for the end of a layer with a weighted sum: pending sublayer output, token input and sum together.
+Without one the token input's matrices are two products with a kernel in front and between, and the
+token input stays pending until the next layer's first norm (:class:`NormedPending`).
 
 ``hyper_connection``: the model has several residual streams x_1 .. x_s instead of one
 (:class:`ResidualStreams`), all equal to the embedding output at the start.  A sublayer reads ``u = sum_s
@@ -30,6 +31,18 @@ import torch
 from .. import ops
 from ..config.specs import TensorSpec
 from .base import Part, StateNeed, register_part
+
+
+class NormedPending:
+    """A pending output that enters the stream with a factor and, mostly, through a norm of its own: ``residual +=
+    scale * rms(sum(terms)) * w`` with ``norm = (w, eps)``, or ``scale * sum(terms)`` (None).  A block that ``takes_normed_pending`` adds it in the launch of its first norm; in front
+    of anything else it is settled by a launch of its own."""
+
+    def __init__(self, terms, scale: float, norm) -> None:
+        self.terms, self.scale, self.norm = terms, scale, norm
+
+    def settle(self, residual: torch.Tensor) -> None:
+        ops.stream_norm(self.terms, self.scale, self.norm, residual, None, None)
 
 
 @register_part("stream", "causal_conv_input")

@@ -606,8 +606,8 @@ def side_gate(product, table, token_ids, out):
     out.copy_((_gelu_tanh(_summed(product)) * table[token_ids.long()].float()).to(out.dtype))
 
 
-def stream_tail(residual, pending, pending_scale, token_ids, side, depth, pending_norm=None):
-    _add_pending(residual, pending, pending_scale, pending_norm)
+def stream_tail(residual, pending, pending_scale, token_ids, side, depth):
+    _add_pending(residual, pending, pending_scale)
     if side is not None:
         table, gate, proj_t, norm, eps = side
         g = _gelu_tanh(residual @ gate.float().T) * table[token_ids.long()].float()

@@ -386,16 +386,6 @@ def test_replay_modes_emulated(name, folders, emulated):
     replay_modes(folder, config, weights, PAGE[name], "float32", "cpu", lengths=(1, 5, 9, 23, 37))
 
 
-def test_the_token_input_as_products_emulated(folders, emulated, monkeypatch):
-    """What long steps do at the end of a layer, here from two tokens on."""
-    from einf_b200.parts.block import PreNormStreamBlock
-
-    monkeypatch.setattr(PreNormStreamBlock, "SIDE_PRODUCT_TOKENS", 2)
-    for name in ("mix", "token_input"):
-        folder, config, weights = folders[name]
-        replay_modes(folder, config, weights, 4, "float32", "cpu", lengths=(1, 6, 19))
-
-
 def test_the_stream_after_every_layer_emulated(folders, emulated):
     from einf_b200.engine.replay import TraceReplayer
 
@@ -409,8 +399,9 @@ def test_the_stream_after_every_layer_emulated(folders, emulated):
 
         def spy(residual, pending, ctx, cache, original=original):
             out = original(residual, pending, ctx, cache)
-            assert out is None
-            seen.append(residual.clone())
+            result = residual.clone()
+            out.settle(result)                  # what the next layer's first norm will add
+            seen.append(result)
             return out
 
         block.forward = spy

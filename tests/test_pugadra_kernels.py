@@ -1,7 +1,6 @@
 """The kernels that came with the Pugadra decoder, each alone against its plain PyTorch statement, at
 sizes other than any model's: the store kernel with its convolution (head by head and in 16-byte pieces),
-the stream's norms in front of and behind a sublayer, the end of a layer with a norm of what is pending,
-the clamped gate, the router's bias, an output gate per element in the attention kernels."""
+the stream's norms in front of and behind a sublayer, the token input's gate, the clamped gate, the router's bias, an output gate per element in the attention kernels."""
 import pytest
 import torch
 
@@ -183,33 +182,6 @@ def test_norms_behind_and_in_front_of_a_sublayer(dev, dtype, tokens, hidden, spl
                     results.append([t for t in (residual, out) if t is not None])
                 for got, want in zip(*results):
                     close(got, want, got.dtype)
-
-
-@pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("tokens, hidden, side", [(1, 64, 16), (9, 200, 12), (160, 896, 64), (1100, 256, 8), (7, 37, 5), (3, 512, 0)])
-@pytest.mark.parametrize("splits", [1, 4])
-def test_end_of_a_layer_with_a_norm_of_what_is_pending(dev, dtype, tokens, hidden, side, splits):
-    from einf_b200 import ops
-
-    gen = torch.Generator().manual_seed(2)
-    vocab = 40
-    pending = torch.randn((splits, tokens, hidden), generator=gen).to(dev)
-    pending = pending if splits > 1 else pending[0].to(dtype)
-    residual = torch.randn((tokens, hidden), generator=gen).to(dev)
-    ids = torch.randint(0, vocab, (tokens,), generator=gen).to(torch.int32).to(dev)
-    post = ((1 + 0.2 * torch.randn(hidden, generator=gen)).to(dev), 1e-5)
-    parts = None
-    if side:
-        parts = (torch.randn((vocab, side), generator=gen).to(dtype).to(dev),
-                 (torch.randn((side, hidden), generator=gen) * hidden ** -0.5).to(dtype).to(dev),
-                 torch.randn((side, hidden), generator=gen).to(dtype).to(dev),
-                 (1 + 0.1 * torch.randn(hidden, generator=gen)).to(dev), 1e-5)
-    results = []
-    for fn in (ops.stream_tail, ref.stream_tail):
-        x = residual.clone()
-        fn(x, [pending], 0.6, ids, parts, None, pending_norm=post)
-        results.append(x)
-    torch.testing.assert_close(results[0], results[1], rtol=2e-4, atol=2e-4)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
