@@ -222,7 +222,7 @@ class PugadraConfig(ModelConfig):
         )
 
     def model_spec(self) -> ModelSpec:
-        layers, schedule = [], []
+        layers, schedule, unused = [], [], {}
         for index, layer in enumerate(self.layers):
             prefix = f"l{index}."
             parts = {
@@ -234,6 +234,8 @@ class PugadraConfig(ModelConfig):
                 parts["feed_forward_norm"] = self._norm(prefix + "norm2")
                 parts["feed_forward"] = self._feed_forward(layer["mlp"], prefix + "mlp.")
                 parts["feed_forward_post_norm"] = self._norm(prefix + "norm2b")
+            else:       # the norms of a feed-forward that is not there
+                unused.update({prefix + name: (self.width,) for name in ("norm2", "norm2b")})
             if self.token_side is not None:
                 dim = int(self.token_side["dim"])
                 parts["token_input"] = PartSpec(
@@ -261,4 +263,5 @@ class PugadraConfig(ModelConfig):
                  "tensor_names": {"weight": "head"}},
                 "",
             ),
+            unused_tensors=unused,
         )

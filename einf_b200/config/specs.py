@@ -85,6 +85,8 @@ class ModelSpec:
     #: number of residual streams of a model whose blocks read and write several of them through
     #: vectors of their own (None: one stream that every sublayer's output is added to)
     streams: int | None = None
+    #: tensors that a checkpoint of the architecture may hold although this model makes no use of them: name -> shape
+    unused_tensors: Mapping[str, tuple[int, ...]] = field(default_factory=dict)
 
     def __post_init__(self) -> None:
         if self.streams is not None and any(entry.add_embedding for entry in self.schedule):

@@ -33,12 +33,14 @@ def _part_specs(model_spec: ModelSpec):
 
 
 def expected_tensors(model_spec: ModelSpec) -> tuple[dict[str, TensorSpec], dict[str, TensorSpec]]:
-    """Checkpoint tensors the model needs, and those it tolerates (a stored copy of a tied matrix)."""
+    """Checkpoint tensors the model needs, and those it tolerates (a stored copy of a tied matrix, what the
+    architecture's configuration names as unused)."""
     expected: dict[str, TensorSpec] = {}
     for category, spec in _part_specs(model_spec):
         for name, tensor_spec in part_class(category, spec.kind).tensor_specs(spec).items():
             expected[checkpoint_name(spec, name)] = tensor_spec
-    optional: dict[str, TensorSpec] = {}
+    optional: dict[str, TensorSpec] = {
+        name: TensorSpec(tuple(shape)) for name, shape in model_spec.unused_tensors.items() if name not in expected}
     head = model_spec.head
     if head.get("tied_to"):
         optional[checkpoint_name(head, "weight")] = TensorSpec((head["vocab_size"], head["hidden_size"]))

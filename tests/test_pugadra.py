@@ -242,7 +242,9 @@ def test_configuration_names_every_tensor_of_the_design(folders):
         loaded = load_config(folder)
         assert isinstance(loaded, PugadraConfig)
         expected, optional = expected_tensors(loaded.model_spec())
-        assert set(expected) == set(weights) and set(optional) == {"head"}, name
+        bare = [index for index, entry in enumerate(config["layers"]) if entry["mlp"] is None]
+        assert set(expected) == set(weights), name
+        assert set(optional) == {"head"} | {f"l{index}.{norm}" for index in bare for norm in ("norm2", "norm2b")}, name
         for key, spec in expected.items():
             assert tuple(spec.shape) == tuple(weights[key].shape), key
 
@@ -328,6 +330,21 @@ def test_random_weights_mode_writes_a_folder_the_loader_takes(tmp_path):
     assert set(tensors) == set(expected)
     assert float(tensors["l0.norm1b"].float().abs().max()) < 0.5                 # around zero
     assert abs(float(tensors["l0.side.norm"].float().mean()) - 1.0) < 0.1        # around one
+
+
+def test_stored_norms_of_a_feed_forward_that_is_not_there_change_nothing(folders, tmp_path):
+    from einf_b200.engine.replay import TraceReplayer
+
+    folder, config, weights = folders["convolution"]
+    more = dict(weights)
+    for name in ("l0.norm2", "l0.norm2b"):
+        more[name] = torch.full((config["width"],), 3.0, dtype=torch.bfloat16)
+    write_folder(tmp_path / "m", config, 0, more)
+    requests = make_requests(config, [9])
+    with emulate_kernels():
+        rows = [trace_tools.run_steps(TraceReplayer(where, "float32", 64, block_len=4, device="cpu"), trace_tools.whole(requests))
+                for where in (folder, tmp_path / "m")]
+    assert all(np.array_equal(rows[0][key], rows[1][key]) for key in rows[0])
 
 
 # ---------------------------------------------------------------------------
