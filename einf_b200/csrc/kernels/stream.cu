@@ -193,7 +193,7 @@ __global__ void conv_rows_state_kernel(const float* __restrict__ h, float* __res
 //   residual[t] += scale * y
 //   out[t] = residual[t] * rsqrt(mean(residual[t]^2) + eps) * weight   (weight null: residual[t] itself; out null: nothing)
 // A team of kTeam threads has a row, kVec groups of four columns a thread, in registers between the two
-// sums of squares: a warp (eight rows a CTA) for many rows, a CTA for few or wide ones.  Loads come
+// sums of squares: a warp (four rows a CTA) for many rows, a CTA for few or wide ones.  Loads come
 // first, without a branch between them (an index past the row is clamped, its value unused), so that
 // a whole row is in flight at once.
 // ---------------------------------------------------------------------------
@@ -677,10 +677,10 @@ extern "C" int einf_stream_norm(const void* pend_a, int a_dtype, int a_splits, l
     if (vectors) {
       // partial sums want every load of a row in flight: a warp a row only where there are none
       if (num_tokens >= 256 && hidden <= 2048 && a_splits <= 1) {
-        const int grid = (num_tokens + 7) / 8;
-        if (hidden <= 1024) EINF_STREAM_NORM(32, 8, grid, 256);
-        if (hidden <= 1536) EINF_STREAM_NORM(32, 12, grid, 256);
-        EINF_STREAM_NORM(32, 16, grid, 256);
+        const int grid = (num_tokens + 3) / 4;
+        if (hidden <= 1024) EINF_STREAM_NORM(32, 8, grid, 128);
+        if (hidden <= 1536) EINF_STREAM_NORM(32, 12, grid, 128);
+        EINF_STREAM_NORM(32, 16, grid, 128);
       }
       if (hidden <= 512) EINF_STREAM_NORM(128, 1, num_tokens, 128);
       if (hidden <= 1024) EINF_STREAM_NORM(256, 1, num_tokens, 256);
