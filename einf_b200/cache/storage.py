@@ -9,7 +9,9 @@ tile the attention kernels stream.  Pages of one group share their numbering
 across the layers of the group, so one block table per request serves them all
 (as the single geometry of the reference does,
 ``src/einf/cache/storage.py:52-85``).  Entries with a state need get
-``[slots, *shape]``, zeroed when a request starts.
+``[slots, *shape]``, zeroed when a request starts; flat state rows of one dtype
+lie end to end in one row per slot (every entry's on a 16-byte border), so that one
+kernel clears them all.
 """
 from __future__ import annotations
 
@@ -39,6 +41,7 @@ class CacheStorage:
         self.num_state_slots = num_state_slots
         self._owned: dict[int, torch.Tensor] = {}
         self._states: dict[int, torch.Tensor] = {}
+        needs: dict[int, StateNeed] = {}
         self.views: list[CacheView] = []
         for index, entry in enumerate(plan.entries):
             need = pages_of(entry.need) if entry.owner == index else None
@@ -64,9 +67,8 @@ class CacheStorage:
                     device=device,
                 )
             if state is not None:
-                if num_state_slots <= 0:
-                    raise ValueError("the model has per-request state but the engine has no state slots")
-                self._states[index] = torch.zeros((num_state_slots, *state.shape), dtype=state.dtype, device=device)
+                needs[index] = state
+        self._allocate_states(needs, num_state_slots, device)
         for index, entry in enumerate(plan.entries):
             view = CacheView(writes=False)
             if pages_of(entry.need) is not None:
@@ -78,13 +80,33 @@ class CacheStorage:
                     view.writes = entry.state_owner == index
             self.views.append(view)
 
-    @property
-    def state_tensors(self) -> list[torch.Tensor]:
-        return list(self._states.values())
+    def _allocate_states(self, needs: dict[int, StateNeed], slots: int, device) -> None:
+        #: the tensors ``[slots, ...]`` that hold all state rows
+        self.state_tensors: list[torch.Tensor] = []
+        if not needs:
+            return
+        if slots <= 0:
+            raise ValueError("the model has per-request state but the engine has no state slots")
+        dtypes = {need.dtype for need in needs.values()}
+        if len(dtypes) > 1 or any(len(need.shape) != 1 for need in needs.values()):
+            for index, need in needs.items():
+                self._states[index] = torch.zeros((slots, *need.shape), dtype=need.dtype, device=device)
+            self.state_tensors = list(self._states.values())
+            return
+        dtype = dtypes.pop()
+        border = max(1, 16 // dtype.itemsize)
+        offsets, row = {}, 0
+        for index, need in needs.items():
+            offsets[index] = row
+            row += -(-need.shape[0] // border) * border
+        rows = torch.zeros((slots, row), dtype=dtype, device=device)
+        for index, need in needs.items():
+            self._states[index] = rows[:, offsets[index]:offsets[index] + need.shape[0]]
+        self.state_tensors = [rows]
 
     def bytes(self) -> int:
         total = 0
-        for owned in list(self._owned.values()) + list(self._states.values()):
+        for owned in list(self._owned.values()) + self.state_tensors:
             for t in (owned if isinstance(owned, tuple) else (owned,)):
                 if t is None:
                     continue

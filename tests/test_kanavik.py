@@ -222,7 +222,8 @@ def test_a_layer_plans_pages_and_one_state_row(folders):
         convs = (2 if made["mlp"] is not None else 1) * (taps - 1) * width
         assert entry.need.state.shape == (convs + right["width"] * right["conv"],)
         assert entry.need.pages.value_size == made["mixer"]["left"]["vdim"]
-    assert runner.num_state_slots == 3 and len(runner.storage.state_tensors) == 4
+    assert runner.num_state_slots == 3 and len(runner.storage.state_tensors) == 1
+    assert len({view.state.data_ptr() for view in runner.storage.views if view.state is not None}) == 4
 
 
 def test_configuration_refuses_what_the_design_does_not_have():

@@ -281,7 +281,8 @@ def test_a_looped_span_runs_in_order_with_a_cache_per_pass(folders):
             assert entry.need.pages.value_size == made["mixer"]["left"]["vdim"]
         else:
             assert isinstance(entry.need, PagedKVNeed) and entry.need.window is None
-    assert runner.num_state_slots == 3 and len(runner.storage.state_tensors) == 4   # three runs of layer 1, layer 3
+    assert runner.num_state_slots == 3 and len(runner.storage.state_tensors) == 1
+    assert len({view.state.data_ptr() for view in runner.storage.views if view.state is not None}) == 4   # three runs of layer 1, layer 3
 
 
 def test_configuration_refuses_what_the_design_does_not_have():
